@@ -50,19 +50,169 @@ from ..ops import _lib, functional as Fn, gemm
 from ..parallel import groups
 
 
-class DecodeEngine:
-    def __init__(self, model, max_batch_size: int, max_seq_length: int,
-                 reduce: str = "auto", use_graph: bool = True, use_pdl: bool = True):
-        cfg = model.config
+class GenerationEngine:
+    """The generation loop every model family shares: device-resident loop state, CUDA-graph
+    capture of the decode step, sampling, EOS handling. A family implements ``_decode_step`` (one
+    token for every row, from ``next_tok`` to the sampler) and ``prefill``."""
+
+    reduce = "local"
+
+    def _init_loop(self, model, device, max_batch_size: int, max_seq_length: int,
+                   use_graph: bool, use_pdl: bool):
         self.model = model
-        self.cfg = cfg
-        self.tp = getattr(model, "tp_size", 1)
-        self.dev = model.output.weight.device
-        assert self.dev.type == "cuda", "DecodeEngine needs a CUDA device"
+        self.cfg = model.config
+        self.dev = device
+        assert self.dev.type == "cuda", f"{type(self).__name__} needs a CUDA device"
         self.use_graph = use_graph
         self.use_pdl = use_pdl
         self.B = max_batch_size
         self.S = (max_seq_length + 7) // 8 * 8
+        dev, B = self.dev, self.B
+        self.seed_dev = torch.zeros(1, dtype=torch.int64, device=dev)
+        self.pos = torch.zeros(1, dtype=torch.int32, device=dev)
+        self.next_tok = torch.zeros(B, dtype=torch.int32, device=dev)
+        self.left_pad = torch.zeros(B, dtype=torch.int32, device=dev)
+        self.seq = torch.zeros(B, self.S, dtype=torch.int32, device=dev)
+        self.eos_flag = torch.zeros(B, dtype=torch.int32, device=dev)
+        self.n_unfinished = torch.zeros(1, dtype=torch.int32, device=dev)
+        self.ticket = torch.zeros(1, dtype=torch.int32, device=dev)
+        self._graphs = {}
+        self.launches_per_step = 0
+
+    # ------------------------------------------------------------------ family hooks
+    def _decode_step(self, B, temperature, top_k, eos_id):
+        raise NotImplementedError
+
+    def prefill(self, prompt, left_pad_mask_pos, temperature, top_k, seed, eos_id):
+        raise NotImplementedError
+
+    def _open_rows(self, B: int) -> None:
+        """Called before a generation of B rows (before the graph is captured)."""
+
+    def _close_rows(self) -> None:
+        """Called once the generation's kernels are enqueued."""
+
+    # ------------------------------------------------------------------ shared pieces
+    def _count(self, n):
+        self.launches_per_step += n
+
+    def _sample(self, logits, B, temperature, top_k, eos_id):
+        """Fused sampler on ``logits`` [B, >= vocab]; advances the position."""
+        Fn.sample(logits, temperature=temperature, top_k=top_k, seed=0, seed_dev=self.seed_dev,
+                  pos=self.pos, next_tok=self.next_tok[:B], seq=self.seq[:B], eos_id=eos_id,
+                  eos_flag=self.eos_flag[:B], n_unfinished=self.n_unfinished, ticket=self.ticket,
+                  advance_pos=True, vocab=self.vocab)
+
+    def _begin(self, prompt, left_pad_mask_pos, seed):
+        """Loop state of a new prompt batch; returns the token ids on the device."""
+        B, T = prompt.shape
+        assert B <= self.B and T < self.S
+        dev = self.dev
+        tok = prompt.to(device=dev, dtype=torch.int32).contiguous()
+        self.seq[:B].zero_()
+        self.seq[:B, :T] = tok
+        self.eos_flag.zero_()
+        self.n_unfinished.fill_(B)
+        self.ticket.zero_()
+        if left_pad_mask_pos is None:
+            self.left_pad.zero_()
+        else:
+            self.left_pad[:B] = left_pad_mask_pos.to(device=dev, dtype=torch.int32)
+        self.pos.zero_()
+        self.seed_dev.fill_(int(seed) & (2 ** 63 - 1))
+        return tok
+
+    def _graph_for(self, key):
+        if key in self._graphs:
+            return self._graphs[key]
+        B, temperature, top_k, eos_id = key
+        # warm up on a side stream (module loading, attribute setting), then capture
+        saved = [t.clone() for t in (self.pos, self.next_tok, self.seq, self.eos_flag,
+                                     self.n_unfinished)]
+        s = torch.cuda.Stream()
+        s.wait_stream(torch.cuda.current_stream())
+        with torch.cuda.stream(s):
+            self._decode_step(*key)
+        torch.cuda.current_stream().wait_stream(s)
+        g = torch.cuda.CUDAGraph()
+        self.launches_per_step = 0
+        # programmatic dependent launch: each kernel's prologue overlaps its predecessor's tail
+        old_pdl = _lib.lib().e2h_set_pdl(1 if self.use_pdl else 0)
+        try:
+            with torch.cuda.graph(g):
+                self._decode_step(*key)
+        finally:
+            _lib.lib().e2h_set_pdl(old_pdl)
+        for t, v in zip((self.pos, self.next_tok, self.seq, self.eos_flag, self.n_unfinished),
+                        saved):
+            t.copy_(v)
+        self._graphs[key] = (g, self.launches_per_step)
+        return self._graphs[key]
+
+    # ------------------------------------------------------------------ generate
+    @torch.no_grad()
+    def generate(self, prompt: torch.Tensor, left_pad_mask_pos: Optional[torch.Tensor],
+                 max_new_tokens: int, temperature: float = 1.0, top_k: Optional[int] = None,
+                 eos_id: Optional[int] = None, seed: int = 0, check_eos_every: int = 32):
+        """Returns (seq [B, T+max_new_tokens] int32 on device, number of decode steps run).
+
+        With an ``eos_id`` the loop stops once every row has produced it; the host looks at the
+        device-side counter only every ``check_eos_every`` steps."""
+        B, T = prompt.shape
+        eos = -1 if eos_id is None else int(eos_id)
+        steps = 0
+        key = (B, float(temperature), int(top_k) if top_k else 0, eos)
+        n_dec = min(max_new_tokens - 1, self.S - T - 1)
+        self._open_rows(B)
+        try:
+            if self.use_graph:
+                # before the prompt: the capture's warm-up step runs on whatever the caches hold
+                # and the prompt then starts every row afresh
+                self.pos.zero_()
+                g, _ = self._graph_for(key)
+            self.prefill(prompt, left_pad_mask_pos, temperature, top_k, seed, eos)
+            for i in range(n_dec):
+                if self.use_graph:
+                    g.replay()
+                else:
+                    self._decode_step(*key)
+                steps += 1
+                if eos >= 0 and (i + 1) % check_eos_every == 0 \
+                        and self.n_unfinished.item() <= 0:
+                    break
+        finally:
+            self._close_rows()
+        if self.reduce == "fused":
+            self.check_status()
+        return self.seq[:B, : T + max_new_tokens], steps
+
+    def check_status(self) -> None:
+        """Raises when a kernel of this device recorded a time-out (a tensor-parallel peer that
+        never signalled): the tokens of that generation are not to be trusted."""
+        code = _lib.read_status(self.dev)
+        if code != 0:
+            raise RuntimeError(f"decode engine: a device-side wait timed out (status {code}); "
+                               "a tensor-parallel peer did not reach the same step")
+
+    def decode_launches(self, key=None) -> int:
+        if key is None and self._graphs:
+            return next(iter(self._graphs.values()))[1]
+        return self._graphs[key][1] if key in self._graphs else 0
+
+    def weight_bytes(self) -> int:
+        return sum(p.numel() * p.element_size()
+                   for p in list(self.model.parameters()) + list(self.model.buffers()))
+
+
+class DecodeEngine(GenerationEngine):
+    """LLaMA-architecture models (``models.model.Transformer``)."""
+
+    def __init__(self, model, max_batch_size: int, max_seq_length: int,
+                 reduce: str = "auto", use_graph: bool = True, use_pdl: bool = True):
+        cfg = model.config
+        self.tp = getattr(model, "tp_size", 1)
+        self._init_loop(model, model.output.weight.device, max_batch_size, max_seq_length,
+                        use_graph, use_pdl)
         blk0 = model.layers[0].attention
         self.n_head, self.n_kv, self.D = blk0.n_head, blk0.n_local_heads, blk0.head_dim
         self.dim = model.tok_embeddings.weight.shape[1]
@@ -135,16 +285,6 @@ class DecodeEngine:
                         if self.reduce == "nccl" else None)
         self.logits_shard = (self.sync.extra((B, self.vocab_local), torch.float32)
                              if self.vocab_parallel else None)
-        self.seed_dev = torch.zeros(1, dtype=torch.int64, device=dev)
-        self.pos = torch.zeros(1, dtype=torch.int32, device=dev)
-        self.next_tok = torch.zeros(B, dtype=torch.int32, device=dev)
-        self.left_pad = torch.zeros(B, dtype=torch.int32, device=dev)
-        self.seq = torch.zeros(B, S, dtype=torch.int32, device=dev)
-        self.eos_flag = torch.zeros(B, dtype=torch.int32, device=dev)
-        self.n_unfinished = torch.zeros(1, dtype=torch.int32, device=dev)
-        self.ticket = torch.zeros(1, dtype=torch.int32, device=dev)
-        self._graphs = {}
-        self.launches_per_step = 0
         self.W = [self._layer_weights(blk) for blk in model.layers]
 
     # ------------------------------------------------------------------ weights
@@ -235,14 +375,8 @@ class DecodeEngine:
             self._count(1)
         else:
             gemm.linear(x, m.output.weight, out=logits)
-        Fn.sample(logits, temperature=temperature, top_k=top_k, seed=0, seed_dev=self.seed_dev,
-                  pos=self.pos, next_tok=self.next_tok[:B], seq=self.seq[:B], eos_id=eos_id,
-                  eos_flag=self.eos_flag[:B], n_unfinished=self.n_unfinished, ticket=self.ticket,
-                  advance_pos=True)
+        self._sample(logits, B, temperature, top_k, eos_id)
         self._count(2)
-
-    def _count(self, n):
-        self.launches_per_step += n
 
     def _layers(self, T: int, sq: int, h, xn, q, att, act, prefill_B: int = 0, sync=None):
         m = self.model
@@ -277,33 +411,6 @@ class DecodeEngine:
         self._layers(B, 1, h, xn, q, att, act, sync=self.sync)
         self._head_sample(xn, B, temperature, top_k, eos_id)
 
-    def _graph_for(self, key):
-        if key in self._graphs:
-            return self._graphs[key]
-        B, temperature, top_k, eos_id = key
-        # warm up on a side stream (module loading, attribute setting), then capture
-        saved = [t.clone() for t in (self.pos, self.next_tok, self.seq, self.eos_flag,
-                                     self.n_unfinished)]
-        s = torch.cuda.Stream()
-        s.wait_stream(torch.cuda.current_stream())
-        with torch.cuda.stream(s):
-            self._decode_step(*key)
-        torch.cuda.current_stream().wait_stream(s)
-        g = torch.cuda.CUDAGraph()
-        self.launches_per_step = 0
-        # programmatic dependent launch: each kernel's prologue overlaps its predecessor's tail
-        old_pdl = _lib.lib().e2h_set_pdl(1 if self.use_pdl else 0)
-        try:
-            with torch.cuda.graph(g):
-                self._decode_step(*key)
-        finally:
-            _lib.lib().e2h_set_pdl(old_pdl)
-        for t, v in zip((self.pos, self.next_tok, self.seq, self.eos_flag, self.n_unfinished),
-                        saved):
-            t.copy_(v)
-        self._graphs[key] = (g, self.launches_per_step)
-        return self._graphs[key]
-
     # ------------------------------------------------------------------ prefill
     @torch.no_grad()
     def prefill(self, prompt: torch.Tensor, left_pad_mask_pos: Optional[torch.Tensor],
@@ -312,20 +419,8 @@ class DecodeEngine:
         first new token into ``seq[:, T]``."""
         m = self.model
         B, T = prompt.shape
-        assert B <= self.B and T < self.S
         dev, bf = self.dev, torch.bfloat16
-        tok = prompt.to(device=dev, dtype=torch.int32).contiguous()
-        self.seq[:B].zero_()
-        self.seq[:B, :T] = tok
-        self.eos_flag.zero_()
-        self.n_unfinished.fill_(B)
-        self.ticket.zero_()
-        if left_pad_mask_pos is None:
-            self.left_pad.zero_()
-        else:
-            self.left_pad[:B] = left_pad_mask_pos.to(device=dev, dtype=torch.int32)
-        self.pos.zero_()
-        self.seed_dev.fill_(int(seed) & (2 ** 63 - 1))
+        tok = self._begin(prompt, left_pad_mask_pos, seed)
         n = B * T
         sync = None
         if self.reduce == "fused":
@@ -360,65 +455,21 @@ class DecodeEngine:
             self.sync_prefill = sp
         return sp
 
-    # ------------------------------------------------------------------ generate
-    @torch.no_grad()
-    def generate(self, prompt: torch.Tensor, left_pad_mask_pos: Optional[torch.Tensor],
-                 max_new_tokens: int, temperature: float = 1.0, top_k: Optional[int] = None,
-                 eos_id: Optional[int] = None, seed: int = 0, check_eos_every: int = 32):
-        """Returns (seq [B, T+max_new_tokens] int32 on device, number of decode steps run).
-
-        With an ``eos_id`` the loop stops once every row has produced it; the host looks at the
-        device-side counter only every ``check_eos_every`` steps."""
-        B, T = prompt.shape
-        eos = -1 if eos_id is None else int(eos_id)
-        self.prefill(prompt, left_pad_mask_pos, temperature, top_k, seed, eos)
-        steps = 0
-        key = (B, float(temperature), int(top_k) if top_k else 0, eos)
-        n_dec = min(max_new_tokens - 1, self.S - T - 1)
-        if self.use_graph:
-            g, _ = self._graph_for(key)
-        for i in range(n_dec):
-            if self.use_graph:
-                g.replay()
-            else:
-                self._decode_step(*key)
-            steps += 1
-            if eos >= 0 and (i + 1) % check_eos_every == 0 and self.n_unfinished.item() <= 0:
-                break
-        if self.reduce == "fused":
-            self.check_status()
-        return self.seq[:B, : T + max_new_tokens], steps
-
-    def check_status(self) -> None:
-        """Raises when a kernel of this device recorded a time-out (a tensor-parallel peer that
-        never signalled): the tokens of that generation are not to be trusted."""
-        code = _lib.read_status(self.dev)
-        if code != 0:
-            raise RuntimeError(f"decode engine: a device-side wait timed out (status {code}); "
-                               "a tensor-parallel peer did not reach the same step")
-
-    def decode_launches(self, key=None) -> int:
-        if key is None and self._graphs:
-            return next(iter(self._graphs.values()))[1]
-        return self._graphs[key][1] if key in self._graphs else 0
-
-    def weight_bytes(self) -> int:
-        return sum(p.numel() * p.element_size()
-                   for p in list(self.model.parameters()) + list(self.model.buffers()))
-
-
 def _freqs(S, D, base, dev):
     from ..ops import reference
     return reference.precompute_freqs_cis(S, D, base, dtype=torch.bfloat16, device=dev)
 
 
-def get_engine(model, batch_size: int, seq_length: int, **kw) -> DecodeEngine:
-    """Engine cached on the model; rebuilt when a larger batch / sequence is requested."""
+def get_engine(model, batch_size: int, seq_length: int, **kw) -> GenerationEngine:
+    """Engine cached on the model (of the family the model names with ``make_engine``); rebuilt when
+    a larger batch / sequence is requested."""
     eng = getattr(model, "_decode_engine", None)
     if eng is None or eng.B < batch_size or eng.S < seq_length:
         if eng is not None:
             del model._decode_engine
             torch.cuda.empty_cache()
-        eng = DecodeEngine(model, batch_size, seq_length, **kw)
+        make = getattr(model, "make_engine", None)
+        eng = make(batch_size, seq_length, **kw) if make else \
+            DecodeEngine(model, batch_size, seq_length, **kw)
         model._decode_engine = eng
     return eng

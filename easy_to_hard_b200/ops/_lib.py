@@ -46,6 +46,52 @@ class GemmParams(C.Structure):
         ("a_tiled", C.c_int),
         ("groupsize", C.c_int), ("qsz", C.c_void_p), ("qsz2", C.c_void_p),
         ("phase_clock", C.c_void_p),
+        ("bias", C.c_void_p), ("act", C.c_int), ("act_from", C.c_int), ("tail_from", C.c_int),
+        ("ldt", C.c_longlong), ("tail", C.c_void_p),
+        ("n_groups", C.c_int), ("group_tmax", C.c_int), ("group_off", C.c_void_p),
+    ]
+
+
+class StreamNormParams(C.Structure):
+    """Mirror of ``StreamNormParams`` (csrc/stream_norm.cu)."""
+
+    _fields_ = [
+        ("x", C.c_void_p), ("tokens", C.c_void_p), ("emb", C.c_void_p), ("lde", C.c_longlong),
+        ("vocab", C.c_int), ("emb_scale", C.c_float), ("y", C.c_void_p), ("ldy", C.c_longlong),
+        ("place", C.c_void_p), ("ew", C.c_void_p), ("top", C.c_int), ("y_rows", C.c_int),
+        ("rows", C.c_void_p), ("x_rows", C.c_int), ("weight", C.c_void_p), ("offset", C.c_float),
+        ("eps", C.c_float), ("out", C.c_void_p), ("ldo", C.c_longlong), ("W", C.c_int),
+        ("col", C.c_void_p), ("left_pad", C.c_void_p), ("pos_out", C.c_void_p),
+        ("status", C.c_void_p),
+    ]
+
+
+class AttnWindowParams(C.Structure):
+    """Mirror of ``AttnWindowParams`` (csrc/attn_window.cu)."""
+
+    _fields_ = [
+        ("act", C.c_void_p), ("ld", C.c_longlong), ("off_q", C.c_int), ("off_k", C.c_int),
+        ("off_v", C.c_int), ("off_g", C.c_int), ("kc", C.c_void_p), ("vc", C.c_void_p),
+        ("pos", C.c_void_p), ("slot", C.c_void_p), ("n", C.c_int), ("slots", C.c_int),
+        ("smax", C.c_int), ("H", C.c_int), ("G", C.c_int), ("dim", C.c_int), ("vdim", C.c_int),
+        ("dimp", C.c_int), ("vdimp", C.c_int), ("rot", C.c_int), ("rot_table", C.c_void_p),
+        ("scale", C.c_float), ("window", C.c_int), ("keep", C.c_int), ("qn", C.c_void_p),
+        ("kn", C.c_void_p), ("eps", C.c_float), ("splits", C.c_int), ("status", C.c_void_p),
+    ]
+
+
+class GlaParams(C.Structure):
+    """Mirror of ``E2hGlaParams`` (csrc/gla.cuh)."""
+
+    _fields_ = [
+        ("act", C.c_void_p), ("ld", C.c_longlong), ("off_q", C.c_int), ("off_k", C.c_int),
+        ("off_v", C.c_int), ("off_g", C.c_int), ("a", C.c_void_p), ("lda", C.c_longlong),
+        ("r", C.c_int), ("w2", C.c_void_p), ("ldw", C.c_longlong), ("b2", C.c_void_p),
+        ("inv_tau", C.c_float), ("qscale", C.c_float), ("eps", C.c_float), ("norm", C.c_void_p),
+        ("state", C.c_void_p), ("slots", C.c_int), ("H", C.c_int), ("dim", C.c_int),
+        ("vdim", C.c_int), ("vp", C.c_int), ("pos", C.c_void_p), ("slot", C.c_void_p),
+        ("n", C.c_int), ("splits", C.c_int), ("seg", C.c_void_p), ("n_seg", C.c_int),
+        ("seg_max", C.c_int), ("logdec", C.c_void_p), ("o", C.c_void_p), ("status", C.c_void_p),
     ]
 
 
@@ -57,6 +103,7 @@ EPI_RESIDUAL = 4
 EPI_ROWMAJOR_F32_ACC = 5
 EPI_ROWMAJOR_BF16 = 6
 EPI_DUAL_STORE = 7
+EPI_RESIDUAL_F32 = 8
 
 _vp, _i, _ll, _f, _ull = C.c_void_p, C.c_int, C.c_longlong, C.c_float, C.c_ulonglong
 
@@ -65,6 +112,15 @@ _SIGNATURES = {
     "e2h_gemm_persistent": [C.POINTER(GemmParams), _vp],
     "e2h_gemm_w8": [C.POINTER(GemmParams), _vp],
     "e2h_gemm_w4": [C.POINTER(GemmParams), _vp],
+    "e2h_gemm_f32": [C.POINTER(GemmParams), _vp],
+    "e2h_stream_norm": [C.POINTER(StreamNormParams), _i, _i, _vp],
+    "e2h_attn_prep": [C.POINTER(AttnWindowParams), _i, _vp],
+    "e2h_attn_window": [C.POINTER(AttnWindowParams), _i, _i, _vp],
+    "e2h_gla_step": [C.POINTER(GlaParams), _i, _vp],
+    "e2h_gla_decay": [C.POINTER(GlaParams), _i, _vp],
+    "e2h_gla_scan": [C.POINTER(GlaParams), _i, _vp],
+    "e2h_gla_out": [C.POINTER(GlaParams), _i, _vp],
+    "e2h_moe_route": [_vp, _ll, _i, _i, _i, _vp, _ll, _i, _vp, _ll, _vp, _vp, _vp, _vp, _i, _vp],
     "e2h_rmsnorm_fwd": [_vp, _vp, _vp, _i, C.POINTER(C.c_void_p), _i, _vp, _vp, _vp, _vp, _i, _i, _f,
                         _vp, _vp, _vp, _vp, _vp],
     "e2h_reduce_residual_norm_bf16": [_vp, C.POINTER(C.c_void_p), _i, _vp, _vp, _vp, _i, _i, _f,

@@ -13,10 +13,39 @@ struct EpiCtx {
   int t0;       // first token column of the 8-column group
 };
 
-// Applies the epilogue to 8 consecutive token columns of one feature.
+// Bias and activation of the plain-store epilogues on N tokens of feature f (f < p.F).
+template <int N>
+__device__ __forceinline__ void bias_act(const E2hGemmParams& p, int f, float* v) {
+  if (p.bias != nullptr) {
+    const float b = p.bias[f];
+#pragma unroll
+    for (int j = 0; j < N; ++j) v[j] += b;
+  }
+  if (p.act == 1 && f >= p.act_from && (p.tail_from <= 0 || f < p.tail_from)) {
+#pragma unroll
+    for (int j = 0; j < N; ++j) {
+      const float r = fmaxf(v[j], 0.f);
+      v[j] = r * r;
+    }
+  }
+}
+__device__ __forceinline__ bool in_tail(const E2hGemmParams& p, int f) {
+  return p.tail_from > 0 && f >= p.tail_from;
+}
+// fp32 columns of a launch whose other features leave as bf16
+template <int N>
+__device__ __forceinline__ void store_tail(const E2hGemmParams& p, int f, int t0, const float* v,
+                                           int t_end) {
+#pragma unroll
+  for (int j = 0; j < N; ++j)
+    if (t0 + j < t_end) p.tail[(long long)(t0 + j) * p.ldt + (f - p.tail_from)] = v[j];
+}
+
+// Applies the epilogue to 8 consecutive token columns of one feature. Tokens from t_end on are
+// masked (p.T, or the end of the group in a grouped product).
 template <bool DUAL>
 __device__ __forceinline__ void epilogue8(const E2hGemmParams& p, int f, int t0, float* v,
-                                          float* v2) {
+                                          float* v2, int t_end) {
   const bool f_ok = f < p.F;
   if (p.scale != nullptr) {
     const float s = f_ok ? p.scale[f] : 0.f;
@@ -31,19 +60,39 @@ __device__ __forceinline__ void epilogue8(const E2hGemmParams& p, int f, int t0,
   switch (p.epi) {
     case E2H_EPI_STORE_BF16: {
       __nv_bfloat16* out = static_cast<__nv_bfloat16*>(p.out);
+      if (!f_ok) break;
+      bias_act<8>(p, f, v);
+      if (in_tail(p, f)) {
+        store_tail<8>(p, f, t0, v, t_end);
+        break;
+      }
 #pragma unroll
       for (int j = 0; j < 8; ++j) {
         const int t = t0 + j;
-        if (f_ok && t < p.T) out[(long long)t * p.ldo + f] = __float2bfloat16_rn(v[j]);
+        if (t < t_end) out[(long long)t * p.ldo + f] = __float2bfloat16_rn(v[j]);
       }
     } break;
     case E2H_EPI_STORE_F32: {
       float* out = static_cast<float*>(p.out);
+      if (!f_ok) break;
+      bias_act<8>(p, f, v);
 #pragma unroll
       for (int j = 0; j < 8; ++j) {
         const int t = t0 + j;
-        if (f_ok && t < p.T) out[(long long)t * p.ldo + f] = v[j];
+        if (t < t_end) out[(long long)t * p.ldo + f] = v[j];
       }
+    } break;
+    case E2H_EPI_RESIDUAL_F32: {
+      float* out = static_cast<float*>(p.out);
+      const float* res = static_cast<const float*>(p.aux);
+      if (!f_ok) break;
+      // loads first: `out` may alias `res`
+      float r[8];
+#pragma unroll
+      for (int j = 0; j < 8; ++j) r[j] = t0 + j < t_end ? res[(long long)(t0 + j) * p.ldo + f] : 0.f;
+#pragma unroll
+      for (int j = 0; j < 8; ++j)
+        if (t0 + j < t_end) out[(long long)(t0 + j) * p.ldo + f] = r[j] + v[j];
     } break;
     case E2H_EPI_RESIDUAL: {
       __nv_bfloat16* out = static_cast<__nv_bfloat16*>(p.out);
@@ -54,12 +103,12 @@ __device__ __forceinline__ void epilogue8(const E2hGemmParams& p, int f, int t0,
 #pragma unroll
       for (int j = 0; j < 8; ++j) {
         const int t = t0 + j;
-        r[j] = (f_ok && t < p.T) ? __bfloat162float(res[(long long)t * p.ldo + f]) : 0.f;
+        r[j] = (f_ok && t < t_end) ? __bfloat162float(res[(long long)t * p.ldo + f]) : 0.f;
       }
 #pragma unroll
       for (int j = 0; j < 8; ++j) {
         const int t = t0 + j;
-        if (f_ok && t < p.T)
+        if (f_ok && t < t_end)
           out[(long long)t * p.ldo + f] = __float2bfloat16_rn(bf16_round(v[j]) + r[j]);
       }
     } break;
@@ -69,7 +118,7 @@ __device__ __forceinline__ void epilogue8(const E2hGemmParams& p, int f, int t0,
 #pragma unroll
         for (int j = 0; j < 8; ++j) {
           const int t = t0 + j;
-          if (f_ok && t < p.T) {
+          if (f_ok && t < t_end) {
             const float g = bf16_round(v[j]);
             const float u = bf16_round(v2[j]);
             out[(long long)t * p.ldo + f] = __float2bfloat16_rn(bf16_round(silu(g)) * u);
@@ -84,7 +133,7 @@ __device__ __forceinline__ void epilogue8(const E2hGemmParams& p, int f, int t0,
 #pragma unroll
         for (int j = 0; j < 8; ++j) {
           const int t = t0 + j;
-          if (f_ok && t < p.T) {
+          if (f_ok && t < t_end) {
             out[(long long)t * p.ldo + f] = __float2bfloat16_rn(v[j]);
             out2[(long long)t * p.ldo2 + f] = __float2bfloat16_rn(v2[j]);
           }
@@ -110,7 +159,7 @@ __device__ __forceinline__ void epilogue8(const E2hGemmParams& p, int f, int t0,
 #pragma unroll
           for (int j = 0; j < 8; ++j) {
             const int t = t0 + j;
-            if (t < p.T) row[t] = p.accumulate ? row[t] + v[j] : v[j];
+            if (t < t_end) row[t] = p.accumulate ? row[t] + v[j] : v[j];
           }
         }
       }
@@ -132,7 +181,7 @@ __device__ __forceinline__ void epilogue8(const E2hGemmParams& p, int f, int t0,
 #pragma unroll
           for (int j = 0; j < 8; ++j) {
             const int t = t0 + j;
-            if (t < p.T) row[t] = __float2bfloat16_rn(v[j]);
+            if (t < t_end) row[t] = __float2bfloat16_rn(v[j]);
           }
         }
       }
@@ -166,7 +215,7 @@ __device__ __forceinline__ void epilogue8(const E2hGemmParams& p, int f, int t0,
         }
         cj[j] = 1.f;
         sj[j] = 0.f;
-        if (!is_v && f_ok && t0 + j < p.T) {
+        if (!is_v && f_ok && t0 + j < t_end) {
           const __nv_bfloat162 cs = freqs2[(long long)posj[j] * (D / 2) + (d >> 1)];
           cj[j] = __bfloat162float(cs.x);
           sj[j] = __bfloat162float(cs.y);
@@ -177,7 +226,7 @@ __device__ __forceinline__ void epilogue8(const E2hGemmParams& p, int f, int t0,
         const int t = t0 + j;
         const float x = bf16_round(v[j]);
         const float partner = __shfl_xor_sync(0xffffffffu, x, 1);
-        if (!(f_ok && t < p.T)) continue;
+        if (!(f_ok && t < t_end)) continue;
         float y = x;
         if (!is_v) y = (d & 1) ? (x * cj[j] + partner * sj[j]) : (x * cj[j] - partner * sj[j]);
         const __nv_bfloat16 yb = __float2bfloat16_rn(y);
@@ -208,7 +257,7 @@ __host__ __device__ inline bool epi_can_stage(const E2hGemmParams& p, int tile_r
   if (p.epi != E2H_EPI_STORE_BF16 && p.epi != E2H_EPI_RESIDUAL && p.epi != E2H_EPI_SWIGLU &&
       p.epi != E2H_EPI_ROPE_KV)
     return false;
-  if ((p.F & 7) || (p.ldo & 7) || (tile_rows & 7)) return false;
+  if ((p.F & 7) || (p.ldo & 7) || (tile_rows & 7) || (p.tail_from & 7)) return false;
   if (reinterpret_cast<uintptr_t>(p.out) & 15) return false;
   if (p.epi == E2H_EPI_RESIDUAL && (reinterpret_cast<uintptr_t>(p.aux) & 15)) return false;
   if (p.epi == E2H_EPI_ROPE_KV &&
@@ -253,7 +302,7 @@ __device__ __forceinline__ RopePre rope_prepare(const E2hGemmParams& p, int f) {
 template <bool DUAL>
 __device__ __forceinline__ void stage8(const E2hGemmParams& p, int f, int t0, float* v, float* v2,
                                        __nv_bfloat16* tile, int tl, int pitch, int row,
-                                       const RopePre* rope = nullptr) {
+                                       const RopePre* rope, int t_end) {
   const bool f_ok = f < p.F;
   if (p.scale != nullptr) {
     const float s = f_ok ? p.scale[f] : 0.f;
@@ -291,7 +340,7 @@ __device__ __forceinline__ void stage8(const E2hGemmParams& p, int f, int t0, fl
         const int pos = rp.pos0 + s_;
         if (++s_ == p.sq) s_ = 0;
         float cj = 1.f, sj = 0.f;
-        if (!rp.is_v && f_ok && t0 + j < p.T && pos < p.smax) {
+        if (!rp.is_v && f_ok && t0 + j < t_end && pos < p.smax) {
           const __nv_bfloat162 cs =
               static_cast<const __nv_bfloat162*>(p.freqs)[(long long)pos * (D / 2) + (rp.d >> 1)];
           cj = __bfloat162float(cs.x);
@@ -303,6 +352,13 @@ __device__ __forceinline__ void stage8(const E2hGemmParams& p, int f, int t0, fl
       }
     }
   } else {
+    if (p.epi == E2H_EPI_STORE_BF16 && f_ok) {
+      bias_act<8>(p, f, v);
+      if (in_tail(p, f)) {
+        if (row >= 0) store_tail<8>(p, f, t0, v, t_end);
+        row = -1;
+      }
+    }
 #pragma unroll
     for (int j = 0; j < 8; ++j) y[j] = v[j];
   }
@@ -316,7 +372,7 @@ __device__ __forceinline__ void stage8(const E2hGemmParams& p, int f, int t0, fl
 // thread's index among the epilogue threads, which have synchronised after stage8.
 __device__ __forceinline__ void flush_tile(const E2hGemmParams& p, const __nv_bfloat16* tile,
                                            int pitch, int f_first, int t_first, int n_tok,
-                                           int tid, int nthreads) {
+                                           int tid, int nthreads, int t_end) {
   const int vpr = pitch >> 3;
   const int total = n_tok * vpr;
   __nv_bfloat16* out = static_cast<__nv_bfloat16*>(p.out);
@@ -325,7 +381,7 @@ __device__ __forceinline__ void flush_tile(const E2hGemmParams& p, const __nv_bf
     const int r = i / vpr;
     const int fv = (i - r * vpr) << 3;
     const int t = t_first + r, f = f_first + fv;
-    if (t >= p.T || f >= p.F) continue;
+    if (t >= t_end || f >= p.F || in_tail(p, f)) continue;
     uint4 val = *reinterpret_cast<const uint4*>(tile + r * pitch + fv);
     __nv_bfloat16* dst = out + (long long)t * p.ldo + f;
     if (p.epi == E2H_EPI_RESIDUAL) {

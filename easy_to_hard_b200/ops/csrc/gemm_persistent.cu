@@ -360,6 +360,10 @@ umma_gemm_persistent_kernel(const __grid_constant__ CUtensorMap tmA,
           const float sc = (p.scale != nullptr && f < p.F) ? p.scale[f] : 1.f;
           const float sc2 = (DUAL && p.scale != nullptr && f < p.F) ? p.scale[p.F + f] : 1.f;
           __nv_bfloat16* so = reinterpret_cast<__nv_bfloat16*>(stage_out + b * kChunkBytes);
+          if constexpr (!DUAL) {
+            if (p.epi == E2H_EPI_STORE_BF16 && (p.bias != nullptr || p.act) && f < p.F)
+              bias_act<kChunkTok>(p, f, v);
+          }
           if (staged == 2) {
             // feature-major output (weight gradients): this lane's 32 values are one 64-byte
             // row of the staging tile; the 16-byte pieces are XOR-swizzled (64B TMA swizzle:
@@ -425,7 +429,8 @@ umma_gemm_persistent_kernel(const __grid_constant__ CUtensorMap tmA,
           if (ok) {
 #pragma unroll
             for (int b8 = 0; b8 < 4; ++b8)
-              epilogue8<DUAL>(p, f, t0 + c + 8 * b8, v + 8 * b8, DUAL ? v2 + 8 * b8 : v2);
+              epilogue8<DUAL>(p, f, t0 + c + 8 * b8, v + 8 * b8, DUAL ? v2 + 8 * b8 : v2,
+                              p.T);
           }
         }
       }
@@ -635,7 +640,9 @@ extern "C" int e2h_gemm_persistent(const E2hGemmParams* pp, void* stream_v) {
   E2hGemmParams p = *pp;
   cudaStream_t stream = static_cast<cudaStream_t>(stream_v);
   if (p.F <= 0 || p.T <= 0 || p.K <= 0) return -1;
-  if (p.splitk > 1 || p.a_tiled) return -3;
+  if (p.splitk > 1 || p.a_tiled || p.n_groups > 0 || p.tail_from) return -3;
+  if (p.scale && (p.bias || p.act)) return -3;
+  if ((p.bias || p.act) && p.epi != E2H_EPI_STORE_BF16 && p.epi != E2H_EPI_STORE_F32) return -3;
   if (p.dual && (p.a_mn_major || p.a2 == nullptr)) return -5;
   if ((p.lda % 8) || (p.ldb % 8) || (p.dual && (p.lda2 % 8))) return -6;
   if (((uintptr_t)p.a & 15) || ((uintptr_t)p.b & 15)) return -7;

@@ -103,7 +103,22 @@ umma_gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant_
   const int a_bytes = TH * kTileK * 2;
   const int stage_bytes = a_bytes * (DUAL ? 2 : 1) + Plan::b_bytes;
   const int f0 = blockIdx.x * TH;
-  const int t0 = blockIdx.y * BN;
+  int t0 = blockIdx.y * BN, t_end = p.T;
+  int fa0 = f0;                                  // row of the weight tile in the A operand
+  if (p.n_groups > 0) {
+    // grouped product: blockIdx.y = (group, token tile of the group); the offsets come from the
+    // predecessor, and a tile past the end of its group has nothing to do (every CTA of a
+    // cluster shares blockIdx.y, so clusters leave as a whole)
+    pdl_launch_dependents();
+    pdl_wait_prior();
+    const int per = (p.group_tmax + BN - 1) / BN;
+    const int g = blockIdx.y / per;
+    t0 = p.group_off[g] + (blockIdx.y - g * per) * BN;
+    t_end = p.group_off[g + 1];
+    fa0 = g * p.F + f0;
+    if (t_end > p.T) t_end = p.T;                // offsets come from device memory
+    if (t0 >= t_end || t0 < 0) return;
+  }
 
   const int kb_total = (p.K + kTileK - 1) / kTileK;
   const int kb_begin = (int)((long long)rank * kb_total / S);
@@ -146,7 +161,7 @@ umma_gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant_
   // weight tiles (weights are never written by a preceding kernel of a PDL chain), the epilogue
   // warps wait before they touch the outputs, the MMA thread touches no global memory.
   pdl_launch_dependents();
-  const bool early_weights = kps > 1;
+  const bool early_weights = kps > 1 && p.n_groups == 0;
   if (!(warp == 0 && lane == 0 && early_weights) && !(warp == 1 && lane == 0)) pdl_wait_prior();
 
   if (warp == 0 && lane == 0) {
@@ -170,8 +185,8 @@ umma_gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant_
         const uint32_t a_dst = tiles0 + it * stage_sz;
         const int kb = kb_begin + it * kps;
         mbar_expect_tx(bar, kps * stage_bytes);
-        tma_load_3d_hint(a_dst, &tmA, 0, f0, kb, bar, pol_a);
-        if (DUAL) tma_load_3d_hint(a_dst + kps * a_bytes, &tmA2, 0, f0, kb, bar, pol_a);
+        tma_load_3d_hint(a_dst, &tmA, 0, fa0, kb, bar, pol_a);
+        if (DUAL) tma_load_3d_hint(a_dst + kps * a_bytes, &tmA2, 0, fa0, kb, bar, pol_a);
       }
       pdl_wait_prior();
       E2H_PHASE(p.phase_clock, 2);
@@ -199,8 +214,8 @@ umma_gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant_
         const int kb = kb_begin + it * kps;
         const uint32_t a_dst = st0;
         mbar_expect_tx(bar, kps * stage_bytes);
-        tma_load_3d_hint(a_dst, &tmA, 0, f0, kb, bar, pol_a);
-        if (DUAL) tma_load_3d_hint(a_dst + kps * a_bytes, &tmA2, 0, f0, kb, bar, pol_a);
+        tma_load_3d_hint(a_dst, &tmA, 0, fa0, kb, bar, pol_a);
+        if (DUAL) tma_load_3d_hint(a_dst + kps * a_bytes, &tmA2, 0, fa0, kb, bar, pol_a);
         tma_load_3d(a_dst + kps * a_bytes * (DUAL ? 2 : 1), &tmB, 0, t0, kb, bar);
         armed = it + 1;
         continue;
@@ -216,8 +231,8 @@ umma_gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant_
           tma_load_2d_hint(a_dst, &tmA, 0, row, bar, pol_a);
           if (DUAL) tma_load_2d_hint(a_dst + a_bytes, &tmA2, 0, row, bar, pol_a);
         } else if (!p.a_mn_major) {
-          tma_load_2d_hint(a_dst, &tmA, k0, f0, bar, pol_a);
-          if (DUAL) tma_load_2d_hint(a_dst + a_bytes, &tmA2, k0, f0, bar, pol_a);
+          tma_load_2d_hint(a_dst, &tmA, k0, fa0, bar, pol_a);
+          if (DUAL) tma_load_2d_hint(a_dst + a_bytes, &tmA2, k0, fa0, bar, pol_a);
         } else {
           tma_load_2d(a_dst, &tmA, f0, k0, bar);
           if (TF == 128) tma_load_2d(a_dst + 8192, &tmA, f0 + 64, k0, bar);
@@ -420,9 +435,10 @@ umma_gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant_
         }
         if (staged) {
           stage8<DUAL>(p, f, t0 + c_begin + c + 8 * b, v + 8 * b, DUAL ? v2 + 8 * b : v2, stile,
-                       c + 8 * b, TH, lane_valid ? lane_row : -1, &rope);
+                       c + 8 * b, TH, lane_valid ? lane_row : -1, &rope, t_end);
         } else {
-          epilogue8<DUAL>(p, f, t0 + c_begin + c + 8 * b, v + 8 * b, DUAL ? v2 + 8 * b : v2);
+          epilogue8<DUAL>(p, f, t0 + c_begin + c + 8 * b, v + 8 * b, DUAL ? v2 + 8 * b : v2,
+                            t_end);
         }
       }
     }
@@ -431,7 +447,8 @@ umma_gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant_
   if (staged && is_epi) {
     asm volatile("bar.sync 1, 256;" ::: "memory");   // the eight epilogue warps
     if (acc_ok)
-      flush_tile(p, stile, TH, f0, t0 + rank * slice, slice, threadIdx.x - 64, 256);
+      flush_tile(p, stile, TH, f0, t0 + rank * slice, slice, threadIdx.x - 64, 256,
+                 t_end);
   }
 
   if (warp == 2 && lane == 0) E2H_PHASE(p.phase_clock, 9);
@@ -530,7 +547,10 @@ static int launch(const E2hGemmParams& p, const CUtensorMap& ta, const CUtensorM
   }
   cudaLaunchConfig_t cfg;
   memset(&cfg, 0, sizeof(cfg));
-  cfg.gridDim = dim3((p.F + th - 1) / th, (p.T + BN - 1) / BN, p.splitk);
+  const int t_tiles = p.n_groups > 0 ? p.n_groups * ((p.group_tmax + BN - 1) / BN)
+                                     : (p.T + BN - 1) / BN;
+  if (t_tiles > 65535) return -13;
+  cfg.gridDim = dim3((p.F + th - 1) / th, t_tiles, p.splitk);
   cfg.blockDim = dim3(kThreads, 1, 1);
   cfg.dynamicSmemBytes = smem;
   cfg.stream = stream;
@@ -566,6 +586,13 @@ extern "C" int e2h_gemm_umma(const E2hGemmParams* pp, void* stream_v) {
   if (kb_total < p.splitk) return -4;
   if (p.dual && (p.a_mn_major || p.a2 == nullptr)) return -5;
   if (p.a_tiled && p.a_mn_major) return -5;
+  if (p.n_groups > 0 && (p.a_tiled || p.a_mn_major || p.b_mn_major || p.group_off == nullptr ||
+                         p.group_tmax <= 0 || p.n_signal != 0))
+    return -5;
+  if ((p.bias || p.act || p.tail_from) && p.epi != E2H_EPI_STORE_BF16 && p.epi != E2H_EPI_STORE_F32)
+    return -5;
+  if (p.tail_from && (p.epi != E2H_EPI_STORE_BF16 || p.tail == nullptr)) return -5;
+  const long long a_rows = (long long)p.F * (p.n_groups > 0 ? p.n_groups : 1);
   if ((p.lda % 8) || (p.ldb % 8) || (p.dual && (p.lda2 % 8))) return -6;  // 16-byte strides for TMA
   if (((uintptr_t)p.a & 15) || ((uintptr_t)p.b & 15)) return -7;
   if (p.tf != 64 && p.tf != 128) p.tf = 128;
@@ -598,10 +625,10 @@ extern "C" int e2h_gemm_umma(const E2hGemmParams* pp, void* stream_v) {
   int r;
   const long long tiled_rows = (long long)((p.F + p.tf - 1) / p.tf) * kb_total * p.tf;
   if (p.kps > 1) {
-    r = make_map3d(&ta, p.a, p.K, p.F, p.lda, p.th, p.kps);
+    r = make_map3d(&ta, p.a, p.K, a_rows, p.lda, p.th, p.kps);
     if (r) return r;
     if (p.dual) {
-      r = make_map3d(&ta2, p.a2, p.K, p.F, p.lda2, p.th, p.kps);
+      r = make_map3d(&ta2, p.a2, p.K, a_rows, p.lda2, p.th, p.kps);
       if (r) return r;
     } else {
       ta2 = ta;
@@ -612,13 +639,13 @@ extern "C" int e2h_gemm_umma(const E2hGemmParams* pp, void* stream_v) {
   if (p.a_tiled)
     r = make_map(&ta, p.a, 64, tiled_rows, 64, p.tf);
   else if (!p.a_mn_major)
-    r = make_map(&ta, p.a, p.K, p.F, p.lda, p.th);
+    r = make_map(&ta, p.a, p.K, a_rows, p.lda, p.th);
   else
     r = make_map(&ta, p.a, p.F, p.K, p.lda, 64);
   if (r) return r;
   if (p.dual) {
     r = p.a_tiled ? make_map(&ta2, p.a2, 64, tiled_rows, 64, p.tf)
-                  : make_map(&ta2, p.a2, p.K, p.F, p.lda2, p.th);
+                  : make_map(&ta2, p.a2, p.K, a_rows, p.lda2, p.th);
     if (r) return r;
   } else {
     ta2 = ta;

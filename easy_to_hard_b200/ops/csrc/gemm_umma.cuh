@@ -17,6 +17,7 @@ enum E2hEpilogue : int {
   E2H_EPI_ROWMAJOR_F32_ACC = 5,  // out[f*ldo + t] (+)= acc  (fp32, weight gradients)
   E2H_EPI_ROWMAJOR_BF16 = 6,     // out[f*ldo + t] = bf16(acc)
   E2H_EPI_DUAL_STORE = 7,   // dual A: out[t*ldo+f] = bf16(acc1), out2[t*ldo2+f] = bf16(acc2)
+  E2H_EPI_RESIDUAL_F32 = 8, // out[t*ldo + f] = aux[t*ldo + f] + acc       (fp32 residual stream)
 };
 
 struct E2hGemmParams {
@@ -67,6 +68,18 @@ struct E2hGemmParams {
   const void* qsz;       // bf16 [K / groupsize][F][2] (scale, zero) of A
   const void* qsz2;      // same for A2 of a dual GEMM
   unsigned long long* phase_clock;  // builds with E2H_PHASE_CLOCK only: 16 time stamps per CTA
+  // several projections of one input in one launch (E2H_EPI_STORE_BF16 / _STORE_F32)
+  const float* bias;     // optional per-feature bias added to acc (after `scale`)
+  int act;               // 1: squared ReLU on the features >= act_from (not on the tail)
+  int act_from;
+  int tail_from;         // > 0: features >= tail_from leave as fp32 in tail[t*ldt + f - tail_from]
+  long long ldt;
+  float* tail;
+  // grouped products (mixture of experts): A holds n_groups matrices of F rows one below the
+  // other; rows group_off[g] .. group_off[g + 1] of B (and of out) belong to matrix g
+  int n_groups;
+  int group_tmax;        // host bound of the rows of one group (sizes the grid)
+  const int* group_off;  // device, n_groups + 1 ascending entries
 };
 
 #ifdef __cplusplus

@@ -465,16 +465,18 @@ umma_gemm_w8_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_consta
         }
         if (staged) {
           stage8<DUAL>(p, f, t0 + c_begin + c + 8 * b, v + 8 * b, DUAL ? v2 + 8 * b : v2, stile,
-                       c + 8 * b, TH, lane_valid ? lane_row : -1, &rope);
+                       c + 8 * b, TH, lane_valid ? lane_row : -1, &rope, p.T);
         } else {
-          epilogue8<DUAL>(p, f, t0 + c_begin + c + 8 * b, v + 8 * b, DUAL ? v2 + 8 * b : v2);
+          epilogue8<DUAL>(p, f, t0 + c_begin + c + 8 * b, v + 8 * b, DUAL ? v2 + 8 * b : v2,
+                            p.T);
         }
       }
     }
   }
   if (staged && is_epi) {
     asm volatile("bar.sync 1, 256;" ::: "memory");   // the eight epilogue warps
-    if (acc_ok) flush_tile(p, stile, TH, f0, t0 + rank * slice, slice, threadIdx.x - 64, 256);
+    if (acc_ok) flush_tile(p, stile, TH, f0, t0 + rank * slice, slice, threadIdx.x - 64, 256,
+                            p.T);
   }
 
   if (p.n_signal != 0) __threadfence();

@@ -14,8 +14,9 @@ from typing import Optional
 import torch
 
 from . import _lib
-from ._lib import (EPI_DUAL_STORE, EPI_RESIDUAL, EPI_ROPE_KV, EPI_ROWMAJOR_BF16,
-                   EPI_ROWMAJOR_F32_ACC, EPI_STORE_BF16, EPI_STORE_F32, EPI_SWIGLU, GemmParams)
+from ._lib import (EPI_DUAL_STORE, EPI_RESIDUAL, EPI_RESIDUAL_F32, EPI_ROPE_KV,
+                   EPI_ROWMAJOR_BF16, EPI_ROWMAJOR_F32_ACC, EPI_STORE_BF16, EPI_STORE_F32,
+                   EPI_SWIGLU, GemmParams)
 
 N_SM = 148
 
@@ -109,8 +110,15 @@ def gemm(a: torch.Tensor, b: torch.Tensor, *, epi: int, out: Optional[torch.Tens
          tiled_shape: Optional[tuple] = None, kps: int = 0,
          signal=None, ticket: Optional[torch.Tensor] = None,
          persistent: Optional[bool] = None, pair: Optional[bool] = None,
-         th: Optional[int] = None) -> None:
-    """Raw launch. Shapes: a is [F, K] (or [K, F] when a_mn_major), b is [T, K] (or [K, T]).
+         th: Optional[int] = None, bias: Optional[torch.Tensor] = None,
+         act_from: Optional[int] = None, tail: Optional[torch.Tensor] = None,
+         tail_from: int = 0, group_off: Optional[torch.Tensor] = None, n_groups: int = 0,
+         group_tmax: int = 0) -> None:
+    """Raw launch. ``bias`` (fp32 [F]), ``act_from`` (squared ReLU on the features from there
+    on), ``tail`` / ``tail_from`` (the features from there on leave as fp32) belong to the plain
+    stores; ``group_off`` (int32 [n_groups + 1], ascending) makes the product grouped: ``a`` holds
+    ``n_groups`` matrices below one another and rows group_off[g] .. group_off[g + 1] of ``b`` are
+    multiplied by matrix g (at most ``group_tmax`` rows each). Shapes: a is [F, K] (or [K, F] when a_mn_major), b is [T, K] (or [K, T]).
     An int8 ``a`` (weight-only quantisation; ``scale`` holds the per-feature scales) streams as
     int8 through the converting kernel for up to 128 tokens and is expanded to a scratch bf16
     matrix first for larger token counts."""
@@ -150,9 +158,24 @@ def gemm(a: torch.Tensor, b: torch.Tensor, *, epi: int, out: Optional[torch.Tens
         T, Kb = b.shape
     assert K == Kb, f"contraction mismatch {K} vs {Kb}"
     dual = a2 is not None
+    if n_groups:
+        assert F % n_groups == 0 and not w8 and not w4
+        F //= n_groups
+        if bn is None:
+            bn = 64 if group_tmax <= 64 else 128 if (group_tmax <= 128 or dual) else 256
+        if splitk is None:
+            # the groups already fill the SMs: K is split only as far as they do not
+            splitk, ctas = 1, -(-F // 128) * min(n_groups, T) * -(-group_tmax // bn)
+            while (splitk < 8 and ctas * splitk * 2 <= N_SM and -(-K // 64) // (splitk * 2) >= 4
+                   and bn % (splitk * 2 * 8) == 0):
+                splitk *= 2
+        if kps <= 0:
+            kps = 1 if (K % 64 or bn > 128) else 2
+        tf, persistent = 128, False
     if (w8 or w4) and bn is None:
         bn = 64 if (T <= 64 or dual) else 128
     auto_tiles = (splitk is None and tf is None and kps <= 0 and th is None and not w8 and not w4
+                  and not n_groups
                   and not a_mn_major and not b_mn_major and tiled_shape is None
                   and K % 64 == 0 and STREAM_TILES)
     bn, splitk, stages, tf, kps = pick_tiles(F, T, K, dual, splitk, bn, stages, tf, kps)
@@ -219,6 +242,16 @@ def gemm(a: torch.Tensor, b: torch.Tensor, *, epi: int, out: Optional[torch.Tens
         p.n_head, p.n_kv, p.head_dim = rope["n_head"], rope["n_kv"], rope["head_dim"]
         p.smax = rope["smax"]
         p.kcache, p.vcache = rope["kcache"].data_ptr(), rope["vcache"].data_ptr()
+    if bias is not None:
+        assert bias.dtype == torch.float32 and bias.numel() >= F
+        p.bias = bias.data_ptr()
+    if act_from is not None:
+        p.act, p.act_from = 1, act_from
+    if tail_from:
+        p.tail_from, p.tail, p.ldt = tail_from, tail.data_ptr(), tail.stride(0)
+    if n_groups:
+        assert group_off.dtype == torch.int32 and group_off.numel() > n_groups
+        p.n_groups, p.group_tmax, p.group_off = n_groups, group_tmax, group_off.data_ptr()
     p.status = _lib.status_word(a.device).data_ptr()
     # more than one token tile: the persistent kernel (double-buffered accumulator, TMA-store
     # epilogue); skinny / split-K shapes: the latency-oriented one-tile-per-CTA kernel
@@ -404,3 +437,83 @@ def linear_wgrad(dy: torch.Tensor, x: torch.Tensor, out: Optional[torch.Tensor] 
     epi = EPI_ROWMAJOR_F32_ACC if out.dtype == torch.float32 else EPI_ROWMAJOR_BF16
     gemm(dy, x, epi=epi, out=out, a_mn_major=True, b_mn_major=True, accumulate=accumulate, **kw)
     return out
+
+
+# ---------------------------------------------------------------------------------------------
+# Products of the hybrid decoders: bf16 operands on the tensor cores, fp32 operands through the
+# true 32-bit kernel (csrc/gemm_f32.cu). The residual stream and the tails are fp32 in both.
+
+def _gemm_f32(a, b, *, epi, out, a2=None, aux=None, bias=None, act_from=None, tail=None,
+              tail_from=0, group_off=None, n_groups=0, group_tmax=0) -> None:
+    assert a.dtype == b.dtype == torch.float32 and a.shape[1] == b.shape[1]
+    p = GemmParams()
+    p.F, p.T, p.K = a.shape[0] // max(n_groups, 1), b.shape[0], a.shape[1]
+    p.epi, p.lda, p.ldb, p.a, p.b = epi, _ld(a), _ld(b), a.data_ptr(), b.data_ptr()
+    if a2 is not None:
+        p.dual, p.a2, p.lda2 = 1, a2.data_ptr(), _ld(a2)
+    p.out, p.ldo = out.data_ptr(), out.stride(0)
+    if aux is not None:
+        assert aux.stride(0) == out.stride(0)
+        p.aux = aux.data_ptr()
+    if bias is not None:
+        p.bias = bias.data_ptr()
+    if act_from is not None:
+        p.act, p.act_from = 1, act_from
+    if tail_from:
+        p.tail_from, p.tail, p.ldt = tail_from, tail.data_ptr(), tail.stride(0)
+    if n_groups:
+        p.n_groups, p.group_tmax, p.group_off = n_groups, group_tmax, group_off.data_ptr()
+    _lib.check(_lib.lib().e2h_gemm_f32(C.byref(p), _lib.stream()), "e2h_gemm_f32")
+
+
+def linear_packed(x, w, out, *, bias=None, act_from=None, tail=None) -> int:
+    """Several projections of x at once: ``out`` [T, F0] takes the first F0 features of ``w`` in
+    x's type (squared ReLU from feature ``act_from`` on), ``tail`` [T, F - F0] the others in fp32;
+    ``bias`` fp32 [F]. Returns the number of launches."""
+    F0, F = out.shape[1], w.shape[0]
+    if x.dtype == torch.float32:
+        _gemm_f32(w, x, epi=EPI_STORE_F32, out=out, bias=bias, act_from=act_from, tail=tail,
+                  tail_from=F0 if F > F0 else 0)
+        return 1
+    if F > F0 and x.shape[0] <= 128:
+        gemm(w, x, epi=EPI_STORE_BF16, out=out, bias=bias, act_from=act_from, tail=tail,
+             tail_from=F0)
+        return 1
+    gemm(w[:F0], x, epi=EPI_STORE_BF16, out=out, bias=bias, act_from=act_from)
+    if F == F0:
+        return 1
+    # many tokens: the few tail features would break the large tiles of the main product
+    gemm(w[F0:], x, epi=EPI_STORE_F32, out=tail, bias=None if bias is None else bias[F0:])
+    return 2
+
+
+def linear_residual_f32(x, w, residual) -> None:
+    """residual (fp32, in place) += x @ w^T."""
+    if x.dtype == torch.float32:
+        _gemm_f32(w, x, epi=EPI_RESIDUAL_F32, out=residual, aux=residual)
+    else:
+        gemm(w, x, epi=EPI_RESIDUAL_F32, out=residual, aux=residual)
+
+
+def linear_f32_out(x, w, out) -> None:
+    """out (fp32) = x @ w^T."""
+    if x.dtype == torch.float32:
+        _gemm_f32(w, x, epi=EPI_STORE_F32, out=out)
+    else:
+        gemm(w, x, epi=EPI_STORE_F32, out=out)
+
+
+def grouped_swiglu(x, w1, w3, out, group_off, n_groups: int, group_tmax: int) -> None:
+    """Rows of group g: silu(x @ w1[g]^T) * (x @ w3[g]^T)."""
+    kw = dict(a2=w3, epi=EPI_SWIGLU, out=out, group_off=group_off, n_groups=n_groups,
+              group_tmax=group_tmax)
+    _gemm_f32(w1, x, **kw) if x.dtype == torch.float32 else gemm(w1, x, **kw)
+
+
+def grouped_linear(x, w, out, group_off, n_groups: int, group_tmax: int) -> None:
+    """Rows of group g: x @ w[g]^T."""
+    kw = dict(out=out, group_off=group_off, n_groups=n_groups, group_tmax=group_tmax)
+    if x.dtype == torch.float32:
+        _gemm_f32(w, x, epi=EPI_STORE_F32, **kw)
+    else:
+        gemm(w, x, epi=EPI_STORE_BF16, **kw)

@@ -1,0 +1,186 @@
+"""Front-ends of the hybrid decoders' kernels: fp32-residual norm, windowed attention over the slot
+cache, gated linear attention, expert routing. All of them take bf16 or fp32 activations; there is
+no CPU path."""
+from __future__ import annotations
+
+import ctypes as C
+from typing import Optional
+
+import torch
+
+from . import _lib
+from ._lib import AttnWindowParams, GlaParams, StreamNormParams
+
+N_SM = 148
+
+
+def _is_bf16(t: torch.Tensor) -> int:
+    assert t.dtype in (torch.bfloat16, torch.float32)
+    return int(t.dtype == torch.bfloat16)
+
+
+def stream_norm(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, *, eps: float,
+                offset: float = 0.0, tokens: Optional[torch.Tensor] = None,
+                emb: Optional[torch.Tensor] = None, emb_scale: float = 1.0,
+                experts: Optional[tuple] = None, rows: Optional[torch.Tensor] = None,
+                col: Optional[torch.Tensor] = None, left_pad: Optional[torch.Tensor] = None,
+                pos_out: Optional[torch.Tensor] = None) -> None:
+    """out = rmsnorm(row) * (offset + weight) for the fp32 residual ``x`` [n, W].
+
+    ``tokens`` starts the stream (x = emb[token] * emb_scale); ``experts`` = (y, place, weights)
+    first adds the weighted expert outputs of the layer before to x; ``rows`` normalises only
+    these rows and leaves x alone. ``col`` / ``left_pad`` / ``pos_out``: positions of a decode
+    step."""
+    n, W = (rows if rows is not None else x).shape[0], x.shape[1]
+    assert x.is_contiguous() and x.dtype == torch.float32 and weight.dtype == torch.float32
+    assert out.stride(1) == 1 and out.shape[0] >= n
+    p = StreamNormParams()
+    p.x, p.W, p.x_rows = x.data_ptr(), W, x.shape[0]
+    if tokens is not None:
+        assert emb.dtype == out.dtype and tokens.dtype == torch.int32 and rows is None
+        p.tokens, p.emb, p.lde = tokens.data_ptr(), emb.data_ptr(), emb.stride(0)
+        p.vocab, p.emb_scale = emb.shape[0], emb_scale
+    if experts is not None:
+        y, place, w = experts
+        assert y.dtype == out.dtype and place.dtype == torch.int32 and w.dtype == torch.float32
+        p.y, p.ldy, p.y_rows = y.data_ptr(), y.stride(0), y.shape[0]
+        p.place, p.ew, p.top = place.data_ptr(), w.data_ptr(), place.shape[1]
+    if rows is not None:
+        p.rows = rows.data_ptr()
+    if col is not None:
+        p.col, p.left_pad, p.pos_out = col.data_ptr(), _lib.ptr(left_pad), pos_out.data_ptr()
+    p.weight, p.offset, p.eps = weight.data_ptr(), offset, eps
+    p.out, p.ldo = out.data_ptr(), out.stride(0)
+    p.status = _lib.status_word(x.device).data_ptr()
+    _lib.check(_lib.lib().e2h_stream_norm(C.byref(p), n, _is_bf16(out), _lib.stream()),
+               "stream_norm")
+
+
+def window_splits(n: int, heads: int, kv_heads: int, keys: int) -> int:
+    """CTAs that share one (token, kv head) of ``attn_window``: enough to fill the SMs a few times
+    over, while each still has some 64 keys."""
+    per_g = heads // kv_heads
+    ctas = n * kv_heads * -(-per_g // 8)
+    s = 1
+    while s < 8 and ctas * s * 2 <= N_SM * 8 and keys // (s * 2) >= 64:
+        s *= 2
+    return s
+
+
+class WindowAttention:
+    """Attention of one layer over the slot cache. ``act`` is the packed activation, ``offs`` the
+    columns of q, k, v and the gate; ``qn`` / ``kn`` are the norm weights over the whole
+    projections (or None)."""
+
+    def __init__(self, mixer, offs, kcache, vcache, rot_table, qn, kn, eps: float):
+        self.m, self.kc, self.vc = mixer, kcache, vcache
+        self.keys = kcache.shape[2] if not mixer.window else min(kcache.shape[2],
+                                                                mixer.window + mixer.keep)
+        p = self.p = AttnWindowParams()
+        p.off_q, p.off_k, p.off_v, p.off_g = offs
+        p.kc, p.vc = kcache.data_ptr(), vcache.data_ptr()
+        p.slots, p.smax, p.dimp, p.vdimp = (kcache.shape[0], kcache.shape[2], kcache.shape[3],
+                                            vcache.shape[3])
+        p.H, p.G, p.dim, p.vdim = mixer.heads, mixer.kv_heads, mixer.dim, mixer.vdim
+        assert rot_table.dtype == torch.float32 and rot_table.is_contiguous()
+        assert rot_table.shape[0] >= p.smax and rot_table.shape[1] * 2 == mixer.rot.dims
+        self.rot_table = rot_table
+        p.rot, p.rot_table = mixer.rot.dims, rot_table.data_ptr()
+        p.scale, p.window, p.keep = mixer.scale, mixer.window, mixer.keep
+        p.qn, p.kn, p.eps = _lib.ptr(qn), _lib.ptr(kn), eps
+        p.status = _lib.status_word(kcache.device).data_ptr()
+
+    def _bind(self, act, pos, slot):
+        p = self.p
+        assert act.dtype == self.kc.dtype and act.stride(1) == 1
+        p.act, p.ld, p.n = act.data_ptr(), act.stride(0), act.shape[0]
+        p.pos, p.slot = pos.data_ptr(), slot.data_ptr()
+        return p
+
+    def decode(self, act, pos, slot) -> None:
+        """One token per sequence: norms, rotation, cache write, attention and gate."""
+        p = self._bind(act, pos, slot)
+        p.splits = window_splits(p.n, p.H, p.G, self.keys)
+        _lib.check(_lib.lib().e2h_attn_window(C.byref(p), 1, _is_bf16(act), _lib.stream()),
+                   "attn_window")
+
+    def prep(self, act, pos, slot) -> None:
+        p = self._bind(act, pos, slot)
+        p.splits = 1
+        _lib.check(_lib.lib().e2h_attn_prep(C.byref(p), _is_bf16(act), _lib.stream()),
+                   "attn_prep")
+
+    def prompt(self, act, pos, slot, seg, n_seg: int, seg_max: int) -> int:
+        """Tokens seg[s] .. seg[s + 1] continue one sequence each. Returns the launches."""
+        self.prep(act, pos, slot)
+        self.from_cache(act, pos, slot)
+        return 2
+
+    def from_cache(self, act, pos, slot) -> None:
+        """Attention of tokens that ``prep`` has put into the cache."""
+        p = self._bind(act, pos, slot)
+        p.splits = window_splits(p.n, p.H, p.G, self.keys)
+        _lib.check(_lib.lib().e2h_attn_window(C.byref(p), 0, _is_bf16(act), _lib.stream()),
+                   "attn_window")
+
+
+class GatedLinearAttention:
+    """Gated linear attention of one layer over the slot states."""
+
+    def __init__(self, mixer, offs, state, a2, a2_b, norm, eps: float):
+        self.m, self.state, self.a2 = mixer, state, a2
+        p = self.p = GlaParams()
+        p.off_q, p.off_k, p.off_v, p.off_g = offs
+        p.r, p.w2, p.ldw, p.b2 = a2.shape[1], a2.data_ptr(), a2.stride(0), a2_b.data_ptr()
+        p.inv_tau, p.qscale, p.eps = 1.0 / mixer.tau, mixer.dim ** -0.5, eps
+        p.norm, p.state = norm.data_ptr(), state.data_ptr()
+        p.slots, p.H, p.dim, p.vdim, p.vp = (state.shape[0], mixer.heads, mixer.dim, mixer.vdim,
+                                             state.shape[3])
+        p.status = _lib.status_word(state.device).data_ptr()
+
+    def _bind(self, act, tail, pos, slot):
+        p = self.p
+        assert act.dtype == self.a2.dtype and tail.dtype == torch.float32
+        p.act, p.ld, p.n = act.data_ptr(), act.stride(0), act.shape[0]
+        p.a, p.lda = tail.data_ptr(), tail.stride(0)
+        p.pos, p.slot = pos.data_ptr(), slot.data_ptr()
+        return p
+
+    def decode(self, act, tail, pos, slot) -> None:
+        p = self._bind(act, tail, pos, slot)
+        s = 1
+        while s < 8 and (p.n * p.H * s * 2 <= N_SM * 4 and p.vp // (s * 2) >= 32
+                         or p.vp // s > 1024):
+            s *= 2
+        p.splits = s
+        _lib.check(_lib.lib().e2h_gla_step(C.byref(p), _is_bf16(act), _lib.stream()), "gla_step")
+
+    def prompt(self, act, tail, pos, slot, seg, n_seg: int, seg_max: int) -> int:
+        """Tokens seg[s] .. seg[s + 1] continue one sequence each. Returns the launches."""
+        p = self._bind(act, tail, pos, slot)
+        n = p.n
+        logdec = torch.empty(n, p.H * p.dim, dtype=torch.float32, device=act.device)
+        o = torch.empty(n, p.H * p.vdim, dtype=torch.float32, device=act.device)
+        p.logdec, p.o = logdec.data_ptr(), o.data_ptr()
+        p.seg, p.n_seg, p.seg_max = seg.data_ptr(), n_seg, seg_max
+        lib, bf, s = _lib.lib(), _is_bf16(act), _lib.stream()
+        _lib.check(lib.e2h_gla_decay(C.byref(p), bf, s), "gla_decay")
+        _lib.check(lib.e2h_gla_scan(C.byref(p), bf, s), "gla_scan")
+        _lib.check(lib.e2h_gla_out(C.byref(p), bf, s), "gla_out")
+        return 3
+
+
+def moe_route(logits: torch.Tensor, experts: int, top: int, h: torch.Tensor, hg: torch.Tensor,
+              off: torch.Tensor, place: torch.Tensor, weights: torch.Tensor,
+              sel: torch.Tensor) -> int:
+    """Top-``top`` routing of fp32 ``logits`` [n, >= experts]: ``weights`` / ``place`` [n, top]
+    (softmax over the chosen logits; row of ``hg`` that holds the token for that choice), ``off``
+    [experts + 1] (rows of every expert), ``hg`` [n * top, W] (h regrouped by expert)."""
+    n = h.shape[0]
+    assert logits.dtype == torch.float32 and hg.dtype == h.dtype and hg.shape[0] >= n * top
+    assert off.numel() > experts and sel.numel() >= n * top
+    _lib.check(_lib.lib().e2h_moe_route(
+        logits.data_ptr(), logits.stride(0), n, experts, top, h.data_ptr(), h.stride(0),
+        h.shape[1], hg.data_ptr(), hg.stride(0), off.data_ptr(), place.data_ptr(),
+        weights.data_ptr(), sel.data_ptr(), _is_bf16(h), _lib.stream()), "moe_route")
+    return 1 if n * top <= 1024 and n <= 256 else 3
