@@ -91,7 +91,9 @@ class GlaParams(C.Structure):
         ("state", C.c_void_p), ("slots", C.c_int), ("H", C.c_int), ("dim", C.c_int),
         ("vdim", C.c_int), ("vp", C.c_int), ("pos", C.c_void_p), ("slot", C.c_void_p),
         ("n", C.c_int), ("splits", C.c_int), ("seg", C.c_void_p), ("n_seg", C.c_int),
-        ("seg_max", C.c_int), ("logdec", C.c_void_p), ("o", C.c_void_p), ("status", C.c_void_p),
+        ("seg_max", C.c_int), ("logdec", C.c_void_p), ("o", C.c_void_p), ("chunks", C.c_int),
+        ("cq", C.c_void_p), ("ck", C.c_void_p), ("ca", C.c_void_p), ("cg", C.c_void_p),
+        ("status", C.c_void_p),
     ]
 
 
@@ -116,6 +118,9 @@ _SIGNATURES = {
     "e2h_stream_norm": [C.POINTER(StreamNormParams), _i, _i, _vp],
     "e2h_attn_prep": [C.POINTER(AttnWindowParams), _i, _vp],
     "e2h_attn_window": [C.POINTER(AttnWindowParams), _i, _i, _vp],
+    "e2h_gla_chunk": [C.POINTER(GlaParams), _vp],
+    "e2h_flash_window": [_vp, _ll, _i, _i, _vp, _vp, _vp, _i, _i, _vp, _vp, _i, _i, _i, _i, _i, _i,
+                         _i, _i, _i, _f, _i, _i, _vp, _vp],
     "e2h_gla_step": [C.POINTER(GlaParams), _i, _vp],
     "e2h_gla_decay": [C.POINTER(GlaParams), _i, _vp],
     "e2h_gla_scan": [C.POINTER(GlaParams), _i, _vp],

@@ -57,10 +57,11 @@ __global__ void __launch_bounds__(kStepThreads) gla_step_kernel(const E2hGlaPara
   const int v0 = rank * vb, nv = max(min(vb, p.vp - v0), 0);
   const int nq4 = vb / 4;                                     // column quads
   const int groups = kStepThreads / nq4 > 0 ? kStepThreads / nq4 : 1;
+  const int dp = (p.dim + 3) / 4 * 4;   // every array starts on a 16-byte boundary
   float* al = gs;                       // [dim] decay
-  float* ks = al + p.dim;               // [dim]
-  float* qs = ks + p.dim;               // [dim]
-  float* as = qs + p.dim;               // [r]
+  float* ks = al + dp;                  // [dim]
+  float* qs = ks + dp;                  // [dim]
+  float* as = qs + dp;                  // [r]
   float* vs = as + (p.r + 3) / 4 * 4;   // [vb]
   float* os = vs + vb;                  // [groups][vb]
   pdl_launch_dependents();
@@ -284,7 +285,7 @@ template <typename T>
 static int step(const E2hGlaParams& p, cudaStream_t stream) {
   const int vb = (p.vp / 4 + p.splits - 1) / p.splits * 4;
   const int groups = kStepThreads / (vb / 4) > 0 ? kStepThreads / (vb / 4) : 1;
-  const size_t smem = 4 * ((size_t)3 * p.dim + (p.r + 3) / 4 * 4 + vb + (size_t)groups * vb);
+  const size_t smem = 4 * ((size_t)3 * ((p.dim + 3) / 4 * 4) + (p.r + 3) / 4 * 4 + vb + (size_t)groups * vb);
   if (smem > 48 * 1024 || vb > 1024) return -2;
   cudaLaunchConfig_t cfg;
   memset(&cfg, 0, sizeof(cfg));

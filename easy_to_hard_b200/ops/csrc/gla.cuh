@@ -33,7 +33,13 @@ struct E2hGlaParams {
   // prompts: segment s holds tokens seg[s] .. seg[s + 1] of one sequence
   const int* seg;          // [n_seg + 1]
   int n_seg, seg_max;      // host bound of a segment's length
-  float* logdec;           // fp32 [n, H * dim] scratch: log alpha
+  float* logdec;           // fp32 [n, H * dim] scratch: log alpha (scan)
   float* o;                // fp32 [n, H * vdim] scratch
+  // chunked form: 64-token chunks, chunk c of segment s in place seg[s] / 64 + s + c
+  int chunks;              // places: n / 64 + n_seg + 1
+  void* cq;                // bf16 [2 (high, low part)][chunks, H, 64, dim]: q e^{b_t}
+  void* ck;                // bf16 [2][chunks, H, 64, dim]: k e^{b_end - b_t}
+  void* ca;                // bf16 [2][chunks, H, 64, 64]: lower-triangular scores in the chunk
+  float* cg;               // fp32 [chunks, H, dim]: e^{b_end}
   int* status;
 };

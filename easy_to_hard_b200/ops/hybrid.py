@@ -72,8 +72,12 @@ class WindowAttention:
     columns of q, k, v and the gate; ``qn`` / ``kn`` are the norm weights over the whole
     projections (or None)."""
 
+    # shortest longest-segment for which the 128-query tensor-core tiles pay
+    TENSOR_CORE_TOKENS = 24
+
     def __init__(self, mixer, offs, kcache, vcache, rot_table, qn, kn, eps: float):
         self.m, self.kc, self.vc = mixer, kcache, vcache
+        self._held = (rot_table, qn, kn)     # the kernels keep raw addresses
         self.keys = kcache.shape[2] if not mixer.window else min(kcache.shape[2],
                                                                 mixer.window + mixer.keep)
         p = self.p = AttnWindowParams()
@@ -84,7 +88,6 @@ class WindowAttention:
         p.H, p.G, p.dim, p.vdim = mixer.heads, mixer.kv_heads, mixer.dim, mixer.vdim
         assert rot_table.dtype == torch.float32 and rot_table.is_contiguous()
         assert rot_table.shape[0] >= p.smax and rot_table.shape[1] * 2 == mixer.rot.dims
-        self.rot_table = rot_table
         p.rot, p.rot_table = mixer.rot.dims, rot_table.data_ptr()
         p.scale, p.window, p.keep = mixer.scale, mixer.window, mixer.keep
         p.qn, p.kn, p.eps = _lib.ptr(qn), _lib.ptr(kn), eps
@@ -113,7 +116,15 @@ class WindowAttention:
     def prompt(self, act, pos, slot, seg, n_seg: int, seg_max: int) -> int:
         """Tokens seg[s] .. seg[s + 1] continue one sequence each. Returns the launches."""
         self.prep(act, pos, slot)
-        self.from_cache(act, pos, slot)
+        p = self.p
+        if (act.dtype == torch.bfloat16 and seg_max >= self.TENSOR_CORE_TOKENS
+                and p.dim % 8 == 0 and p.vdim % 8 == 0 and p.dim <= 128 and p.vdim <= 128):
+            _lib.check(_lib.lib().e2h_flash_window(
+                p.act, p.ld, p.off_q, p.off_g, p.kc, p.vc, seg.data_ptr(), n_seg, seg_max, p.pos,
+                p.slot, p.n, p.slots, p.smax, p.H, p.G, p.dim, p.vdim, p.dimp, p.vdimp, p.scale,
+                p.window, p.keep, p.status, _lib.stream()), "flash_window")
+        else:
+            self.from_cache(act, pos, slot)
         return 2
 
     def from_cache(self, act, pos, slot) -> None:
@@ -127,8 +138,12 @@ class WindowAttention:
 class GatedLinearAttention:
     """Gated linear attention of one layer over the slot states."""
 
+    # shortest longest-segment for which the chunked tensor-core form pays
+    CHUNK_TOKENS = 48
+
     def __init__(self, mixer, offs, state, a2, a2_b, norm, eps: float):
         self.m, self.state, self.a2 = mixer, state, a2
+        self._held = (a2_b, norm)            # the kernels keep raw addresses
         p = self.p = GlaParams()
         p.off_q, p.off_k, p.off_v, p.off_g = offs
         p.r, p.w2, p.ldw, p.b2 = a2.shape[1], a2.data_ptr(), a2.stride(0), a2_b.data_ptr()
@@ -159,11 +174,25 @@ class GatedLinearAttention:
         """Tokens seg[s] .. seg[s + 1] continue one sequence each. Returns the launches."""
         p = self._bind(act, tail, pos, slot)
         n = p.n
-        logdec = torch.empty(n, p.H * p.dim, dtype=torch.float32, device=act.device)
-        o = torch.empty(n, p.H * p.vdim, dtype=torch.float32, device=act.device)
-        p.logdec, p.o = logdec.data_ptr(), o.data_ptr()
+
+        def buf(*shape, dtype=torch.float32):
+            return torch.empty(*shape, dtype=dtype, device=act.device)
+        o = buf(n, p.H * p.vdim)
+        p.o = o.data_ptr()
         p.seg, p.n_seg, p.seg_max = seg.data_ptr(), n_seg, seg_max
         lib, bf, s = _lib.lib(), _is_bf16(act), _lib.stream()
+        if (bf and seg_max >= self.CHUNK_TOKENS and p.dim % 16 == 0 and p.dim <= 128
+                and p.vdim % 8 == 0 and p.r <= 128):
+            p.chunks = n // 64 + n_seg + 1
+            cq, ck = (buf(2, p.chunks, p.H, 64, p.dim, dtype=torch.bfloat16) for _ in "qk")
+            ca = buf(2, p.chunks, p.H, 64, 64, dtype=torch.bfloat16)
+            cg = buf(p.chunks, p.H, p.dim)
+            p.cq, p.ck, p.ca, p.cg = (t.data_ptr() for t in (cq, ck, ca, cg))
+            _lib.check(lib.e2h_gla_chunk(C.byref(p), s), "gla_chunk")
+            _lib.check(lib.e2h_gla_out(C.byref(p), bf, s), "gla_out")
+            return 3
+        logdec = buf(n, p.H * p.dim)
+        p.logdec = logdec.data_ptr()
         _lib.check(lib.e2h_gla_decay(C.byref(p), bf, s), "gla_decay")
         _lib.check(lib.e2h_gla_scan(C.byref(p), bf, s), "gla_scan")
         _lib.check(lib.e2h_gla_out(C.byref(p), bf, s), "gla_out")

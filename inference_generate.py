@@ -11,6 +11,9 @@ data-parallel ranks, and appends ``{idx, sample_idx, prompt, output}`` lines to 
 under an exclusive ``flock`` (tensor-parallel rank 0 of each group writes). ``--resume_generation``
 skips the (idx, sample) pairs already present in the output file.
 
+``--checkpoint_path DIR/model.safetensors`` with a ``DIR/config.json`` that names a hybrid design
+(``models.hybrid``: Bovinex) runs that design; everything else stays the same.
+
 On CUDA, ``generate`` runs on the ``DecodeEngine`` (CUDA-graph decode over the sm_100a kernels,
 static KV cache sized to prompt + new tokens instead of the whole ``block_size``); ``--compile``
 is accepted for compatibility and selects the same engine.
@@ -35,6 +38,7 @@ from easy_to_hard_b200.models.rl_model import generate_tokens
 from easy_to_hard_b200.models.tokenizer_utils import AcceleraTokenizer, batch_encode_tokens
 from easy_to_hard_b200.models.tp import (apply_tp, get_data_parallel_rank,
                                          get_data_parallel_world_size, get_model_parallel_rank,
+                                         get_model_parallel_world_size,
                                          initialize_model_parallel, maybe_init_dist)
 
 
@@ -61,7 +65,16 @@ def generate(model: Transformer, prompt: torch.Tensor, left_pad_mask_pos: Option
 
 def _load_model(checkpoint_path: Path, device, precision, use_tp: bool) -> Transformer:
     """Meta-device build, quantised layouts picked from the file name (``int8`` /
-    ``int4.g{G}``), mmap load, tensor-parallel sharding, move to the device."""
+    ``int4.g{G}``), mmap load, tensor-parallel sharding, move to the device. A folder whose
+    ``config.json`` names a registered hybrid design loads as that design instead."""
+    from easy_to_hard_b200.models.hybrid import config_in, load_hybrid
+    if config_in(checkpoint_path.parent) is not None:
+        if torch.device(device).type != "cuda":
+            raise RuntimeError("hybrid decoders run on CUDA devices only")
+        if use_tp and get_model_parallel_world_size() > 1:
+            raise ValueError("hybrid decoders are not tensor-parallel: launch with "
+                             "--tensor_parallel_size 1 (ranks then share the prompts)")
+        return load_hybrid(checkpoint_path.parent, device, precision)
     with torch.device("meta"):
         model = Transformer.from_name(checkpoint_path.parent.name, freeze_tok_embeddings=True,
                                       freeze_output=True, freeze_norm=True)
@@ -162,6 +175,9 @@ def main(seed: int, prompt_file: Path, output_file: Path, batch_size: int = 4,
 
     t0 = time.time()
     model = _load_model(checkpoint_path, device, precision, use_tp)
+    hybrid = hasattr(model, "make_engine")
+    if hybrid and (finetune_checkpoint_path is not None or on_the_fly_8bit_quantization):
+        raise ValueError("hybrid decoders have no finetune checkpoints and no 8-bit weights")
     if finetune_checkpoint_path is not None:
         from easy_to_hard_b200.utils.checkpoint_utils import (get_latest_checkpoint_path,
                                                               load_inference_checkpoint)

@@ -108,6 +108,26 @@ def speculative_decode(model, draft_model, cur_token: torch.Tensor, input_pos: i
     return torch.cat([draft_tokens[:n_ok], multinomial_sample_one_no_sync(new)])
 
 
+def _stream_hybrid(model, prompt: torch.Tensor, max_new_tokens: int, callback,
+                   **sampling_kwargs) -> torch.Tensor:
+    """Token by token on the engine's step function, with the callback after every token."""
+    from easy_to_hard_b200.models.engine import get_engine
+    eng = get_engine(model, 1, prompt.numel() + max_new_tokens)
+    key = object()
+    eng.open(key)
+    try:
+        seq, ids = prompt.tolist(), prompt.tolist()
+        for _ in range(max_new_tokens):
+            logits = eng.step([(key, ids, [len(ids) - 1])])
+            nxt = sample(logits[None], **sampling_kwargs)[0]
+            callback(nxt)
+            ids = nxt.view(-1).tolist()
+            seq += ids
+    finally:
+        eng.close(key)
+    return torch.tensor(seq, dtype=prompt.dtype, device=prompt.device)
+
+
 @torch.no_grad()
 def generate(model: Transformer, prompt: torch.Tensor, max_new_tokens: int, *, interactive: bool,
              draft_model: Optional[Transformer], speculate_k: int = 8, callback=lambda x: x,
@@ -130,6 +150,12 @@ def generate(model: Transformer, prompt: torch.Tensor, max_new_tokens: int, *, i
                               sampling_kwargs.get("top_k"), None,
                               seed=int(torch.randint(0, 2 ** 31 - 1, (1,)).item()))
         return seq[0].to(dtype), {"accept_counts": accept_counts}
+    if hasattr(model, "make_engine"):
+        if speculative:
+            raise ValueError("speculative decoding rewinds the target model, which a recurrent "
+                             "state cannot do")
+        return _stream_hybrid(model, prompt, max_new_tokens, callback, **sampling_kwargs), \
+            {"accept_counts": accept_counts}
     model.setup_caches(max_batch_size=1, max_seq_length=max_seq)
     if speculative and draft_model is not model:
         draft_model.setup_caches(max_batch_size=1, max_seq_length=max_seq)
