@@ -55,8 +55,12 @@ def parse():
     ap.add_argument("--steps", type=int, default=3)
     ap.add_argument("--warmup", type=int, default=3)
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
-    ap.add_argument("--workload", default="decode", choices=["decode", "sft", "prm"],
-                    help="decode: batched generation (headline); sft: full-parameter SFT step")
+    ap.add_argument("--workload", default="decode", choices=["decode", "sft", "prm",
+                                                                       "bovinex"],
+                    help="decode: batched generation (headline); sft: full-parameter SFT step; "
+                    "bovinex: prefill and decode throughput of the hybrid decoder beside the LLaMA "
+                    "path at equal size")
+    ap.add_argument("--size", default="4k", choices=["2k", "4k"], help="bovinex: layer shapes")
     ap.add_argument("--quant", default="none", choices=["none", "int8", "int4"],
                     help="decode: weight-only quantisation of the linears (int4: groups of 128)")
     ap.add_argument("--micro", type=int, default=16, help="sft: sequences per micro batch")
@@ -597,6 +601,94 @@ def run_ours_prm(a):
         print(json.dumps(out), flush=True)
 
 
+HYBRID_BATCH, HYBRID_PROMPT, HYBRID_DECODE, HYBRID_LAYERS = 64, 1024, 64, 8
+
+
+def run_bovinex(a):
+    """Prefill and decode throughput of the Bovinex hybrid decoder (8 layers of the named size,
+    random weights) and of the LLaMA path at equal size (same width, heads, layers and active
+    feed-forward parameters), both through their engines: a step is one batch of 64 prompts of
+    1024 tokens, then 64 captured decode steps. ``value`` = Bovinex decode tokens/s; the e2e number
+    is the same generation through inference_generate.generate with host inputs and outputs."""
+    import torch
+    rank, local, world = dist_setup(a.gpus)
+    if world > 1:
+        raise SystemExit("the bovinex workload runs on one GPU")
+    sys.path.insert(0, os.path.join(ROOT, "bench"))
+    import hybrid_shapes
+    import inference_generate as api
+    from easy_to_hard_b200.models.engine import get_engine
+    from easy_to_hard_b200.ops import _lib
+    B, P, N = HYBRID_BATCH, HYBRID_PROMPT, HYBRID_DECODE
+    gen = torch.Generator().manual_seed(7)
+    host = [torch.randint(0, 32000, (B, P), generator=gen, dtype=torch.int32).pin_memory()
+            for _ in range(a.steps + a.warmup)]
+    host_out = torch.empty(B, P + N + 1, dtype=torch.int32).pin_memory()
+    sampler, res, launches = ClockSampler(local), {}, 0
+    sampler.start()
+    for name in ("bovinex", "llama"):
+        build = getattr(hybrid_shapes, f"{name}_model")
+        model = build(a.size, HYBRID_LAYERS)
+        eng = get_engine(model, B, P + N + 8)
+        dev = [h.cuda() for h in host]
+        key = (B, TEMPERATURE, TOP_K, -1)
+        eng._open_rows(B)
+        eng.pos.zero_()
+        g, per_step = eng._graph_for(key)
+
+        def prefill(i):
+            eng.prefill(dev[i % len(dev)], None, TEMPERATURE, TOP_K, i, -1)
+
+        def decode(i):
+            for _ in range(N):
+                g.replay()
+        for i in range(a.warmup):
+            prefill(i)
+            decode(i)
+        pre = dec = 0.0
+        for i in range(a.steps):
+            pre += timed(prefill, 1)
+            dec += timed(decode, 1)
+        eng._close_rows()
+        res[name] = {"prefill_tokens_per_s": B * P * a.steps / (pre / 1e3),
+                     "decode_tokens_per_s": B * N * a.steps / (dec / 1e3),
+                     "prefill_ms": pre / a.steps, "decode_step_us": dec / a.steps / N * 1e3,
+                     "launches_per_decode_step": per_step,
+                     "weight_bytes": eng.weight_bytes()}
+        if name == "bovinex":
+            launches = (eng.prefill_launches + N * per_step) * a.steps
+
+            def e2e(i):
+                p = host[i % len(host)].to("cuda", non_blocking=True)
+                seq, _ = api.generate(model, p, None, N + 1, temperature=TEMPERATURE, top_k=TOP_K,
+                                      seed=i)
+                host_out.copy_(seq, non_blocking=True)
+                torch.cuda.current_stream().synchronize()
+            e2e(0)
+            ms_e2e = timed(e2e, a.steps)
+        eng._graphs.clear()
+        model._decode_engine = None
+        del model, eng, g
+        torch.cuda.empty_cache()
+    clocks = sampler.stop()
+    b = res["bovinex"]
+    print(json.dumps({
+        "metric": "bovinex_decode_tokens_per_s", "value": b["decode_tokens_per_s"],
+        "unit": "tokens/s", "n_gpus": 1, "steps": a.steps, "warmup": a.warmup,
+        "ms_per_step": b["prefill_ms"] + b["decode_step_us"] * N / 1e3, "higher_is_better": True,
+        "scaling": "strong", "vs_baseline": None, "dtype": "bf16",
+        "data": "synthetic (random token ids, random-init weights)", "impl": "ours",
+        "config": {"model": f"Bovinex {a.size}: {HYBRID_LAYERS} layers, attention / gated linear "
+                            "attention, dense / 8 experts top 2 (bench/hybrid_shapes.py)",
+                   "global_batch": B, "seq_len": P + N, "prompt_len": P, "decode_steps": N,
+                   "parallelism": "tp1",
+                   "l2": "inputs larger than L2 (weights and caches stream per step)"},
+        "bovinex": b, "llama_equal_size": res["llama"], "clocks": clocks,
+        "e2e": {"value": B * (N + 1) * a.steps / (ms_e2e / 1e3), "unit": "tokens/s",
+                "h2d_bytes_per_step": B * P * 4, "d2h_bytes_per_step": B * (P + N + 1) * 4},
+        "gpu_launches": launches, "kernel_status": _lib.read_status()}), flush=True)
+
+
 def run_reference(a):
     """The unmodified reference on the same workload: its own generate() for decode, its own
     training step (FSDP1, its AdamW, its tensor-parallel hooks) for SFT."""
@@ -614,6 +706,8 @@ def run_reference(a):
         from baseline import reference_runner, reference_sft_runner
     except Exception as e:  # noqa: BLE001
         return unavailable(f"reference runner import failed: {type(e).__name__}: {e}")
+    if a.workload == "bovinex":
+        return unavailable("the reference has no such model")
     if a.workload == "prm":
         return unavailable("no reference arm is wired for the reward-model training workload")
     try:
@@ -637,6 +731,8 @@ if __name__ == "__main__":
         run_ours_sft(args)
     elif args.workload == "prm":
         run_ours_prm(args)
+    elif args.workload == "bovinex":
+        run_bovinex(args)
     else:
         run_ours(args)
     finish()

@@ -11,7 +11,7 @@
 // columns hold zeros).
 //
 //   attn_prep    prompts: norms and rotates q and k of every token in place, writes k and v to the
-//                cache. One CTA per token.
+//                cache. One CTA per token (a vectorised form for sizes in multiples of 8).
 //   attn_window  one (token, kv head) per cluster of CTAs: the visible keys are split over the CTAs
 //                of the cluster and merged through distributed shared memory. In its fused form
 //                (decode) it does the work of attn_prep itself, so that a decode step has one
@@ -87,6 +87,104 @@ __device__ __forceinline__ float rms_of(const T* x, int n, float eps, float* red
   }
   ss = block_sum(ss, red);
   return 1.f / sqrtf(ss / n + eps);
+}
+
+// 16-byte-vectorised form: head sizes and half the rotated width are multiples of 8, rows aligned.
+// A thread takes 8 columns of a pair's first halves together with the 8 of the second halves (or 16
+// unrotated columns), twice: once for the sums of squares, once (from L1) to write.
+template <typename T>
+__global__ void __launch_bounds__(128) attn_prep_vec_kernel(const AttnWindowParams p) {
+  __shared__ float red[2][4];
+  pdl_launch_dependents();
+  pdl_wait_prior();
+  const int t = blockIdx.x;
+  const int pos = p.pos[t], slot = p.slot[t];
+  if (pos < 0 || pos >= p.smax || slot < 0 || slot >= p.slots) {
+    if (threadIdx.x == 0) atomicCAS(p.status, 0, kStatusBadArgs);
+    return;
+  }
+  T* row = static_cast<T*>(p.act) + t * p.ld;
+  T* q = row + p.off_q;
+  const T* k = row + p.off_k;
+  const T* v = row + p.off_v;
+  const int vq = p.H * p.dim / 8, vk = p.G * p.dim / 8;
+  float rq = 1.f, rk = 1.f;
+  if (p.qn || p.kn) {
+    float sq = 0.f, sk = 0.f;
+    for (int i = threadIdx.x; i < vq + vk; i += 128) {
+      float x[8], ss = 0.f;
+      load8(i < vq ? q + 8 * i : k + 8 * (i - vq), x);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) ss += x[e] * x[e];
+      if (i < vq) sq += ss;
+      else sk += ss;
+    }
+    sq = warp_sum(sq);
+    sk = warp_sum(sk);
+    if ((threadIdx.x & 31) == 0) {
+      red[0][threadIdx.x >> 5] = sq;
+      red[1][threadIdx.x >> 5] = sk;
+    }
+    __syncthreads();
+    sq = red[0][0] + red[0][1] + red[0][2] + red[0][3];
+    sk = red[1][0] + red[1][1] + red[1][2] + red[1][3];
+    if (p.qn) rq = 1.f / sqrtf(sq / (p.H * p.dim) + p.eps);
+    if (p.kn) rk = 1.f / sqrtf(sk / (p.G * p.dim) + p.eps);
+  }
+  const int half = p.rot >> 1;
+  const int up = half / 8, ur = (p.dim - p.rot) / 8, per = up + ur;   // work units of a head
+  const float* cs = p.rot_table + (long long)pos * p.rot;
+  T* kc = static_cast<T*>(p.kc) + ((long long)slot * p.G * p.smax + pos) * p.dimp;
+  for (int i = threadIdx.x; i < (p.H + p.G) * per; i += 128) {
+    const int head = i / per, u = i - head * per;
+    const bool is_q = head < p.H;
+    const int hk = head - p.H;
+    const T* src = is_q ? q + head * p.dim : k + hk * p.dim;
+    const float* w = is_q ? (p.qn ? p.qn + head * p.dim : nullptr)
+                          : (p.kn ? p.kn + hk * p.dim : nullptr);
+    const float r = is_q ? rq : rk;
+    T* dst = is_q ? q + head * p.dim : kc + (long long)hk * p.smax * p.dimp;
+    auto fetch = [&](int d, float* x) {
+      load8(src + d, x);
+      if (w) {
+        float wv[8];
+        load8(w + d, wv);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) x[e] *= r * wv[e];
+      }
+    };
+    if (u < up) {
+      const int d = 8 * u;
+      float a[8], b[8], c[16];
+      fetch(d, a);
+      fetch(half + d, b);
+      load8(cs + 2 * d, c);
+      load8(cs + 2 * d + 8, c + 8);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) {
+        const float co = c[2 * e], si = c[2 * e + 1], x = a[e], y = b[e];
+        a[e] = x * co - y * si;
+        b[e] = y * co + x * si;
+      }
+      store4(dst + d, a);
+      store4(dst + d + 4, a + 4);
+      store4(dst + half + d, b);
+      store4(dst + half + d + 4, b + 4);
+    } else {
+      const int d = p.rot + 8 * (u - up);
+      float a[8];
+      fetch(d, a);
+      store4(dst + d, a);
+      store4(dst + d + 4, a + 4);
+    }
+  }
+  T* vc = static_cast<T*>(p.vc) + ((long long)slot * p.G * p.smax + pos) * p.vdimp;
+  const int vv = p.vdim * (int)sizeof(T) / 16;               // 16-byte pieces of a value head
+  for (int i = threadIdx.x; i < p.G * vv; i += 128) {
+    const int head = i / vv, c = i - head * vv;
+    reinterpret_cast<uint4*>(vc + (long long)head * p.smax * p.vdimp)[c] =
+        reinterpret_cast<const uint4*>(v + head * p.vdim)[c];
+  }
 }
 
 template <typename T>
@@ -421,6 +519,15 @@ extern "C" int e2h_attn_prep(const e2h::AttnWindowParams* p, int is_bf16, void* 
   using namespace e2h;
   int r = win_check(*p);
   if (r) return r;
+  const bool vec = p->dim % 8 == 0 && p->vdim % 8 == 0 && p->rot % 16 == 0 && p->ld % 8 == 0 &&
+                   p->off_q % 8 == 0 && p->off_k % 8 == 0 && p->off_v % 8 == 0 &&
+                   !((reinterpret_cast<uintptr_t>(p->act) | reinterpret_cast<uintptr_t>(p->qn) |
+                      reinterpret_cast<uintptr_t>(p->kn)) & 15);
+  if (vec)
+    return is_bf16 ? (int)launch(attn_prep_vec_kernel<__nv_bfloat16>, dim3(p->n), dim3(128), 0,
+                                 (cudaStream_t)stream, *p)
+                   : (int)launch(attn_prep_vec_kernel<float>, dim3(p->n), dim3(128), 0,
+                                 (cudaStream_t)stream, *p);
   const size_t smem = (size_t)(p->H + p->G) * p->dim * 4;
   if (smem > 200 * 1024) return -2;
   static std::once_flag once;

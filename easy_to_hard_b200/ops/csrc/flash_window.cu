@@ -317,6 +317,16 @@ flash_window_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
       if (lane == 0) mbar_arrive(smem_u32(&ctrl->p_full));
     }
     // ---- epilogue: O / l * sigmoid(gate) ----
+    // the gate row first, all pieces in flight at once, while the last product finishes
+    const bool in_seq = q0 + row < len;
+    __nv_bfloat16* grow = p.gate + (long long)(t_begin + q0 + row) * p.ld + (long long)h * p.vdim +
+                          ch * DH;
+    const int n_col = min(DH, p.vdim - ch * DH);      // live columns of this thread (may be <= 0)
+    uint4 gr[DH / 8];
+#pragma unroll
+    for (int i = 0; i < DH / 8; ++i)
+      gr[i] = in_seq && i * 8 < n_col ? *reinterpret_cast<const uint4*>(grow + i * 8)
+                                      : make_uint4(0, 0, 0, 0);
     if (ok) ok = mbar_wait(smem_u32(&ctrl->o_full), (n_j - 1) & 1, abort_flag, p.status,
                            kStatusTimeoutTmemFull);
     ok = __all_sync(0xffffffffu, ok);
@@ -325,27 +335,25 @@ flash_window_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
     pair_bar_sync(1 + qrt);
     const float l_tot = l + xch[(ch ^ 1) * 128 + row];
     const float inv = l_tot > 0.f ? 1.f / l_tot : 0.f;
-    const bool store = ok && q0 + row < len;
-    __nv_bfloat16* grow = p.gate + (long long)(t_begin + q0 + row) * p.ld + (long long)h * p.vdim;
+    const bool store = ok && in_seq;
 #pragma unroll
     for (int c = 0; c < DH; c += 32) {
       float ov[32];
       if (ok) tmem_ld_x32(tmem_o + lane_off + ch * DH + c, ov);   // warp-uniform
       tmem_ld_wait();
-      if (!store) continue;
 #pragma unroll
-      for (int c8 = 0; c8 < 32; c8 += 8) {
-        const int col = ch * DH + c + c8;
-        if (col >= p.vdim) continue;
-        uint4 gr = *reinterpret_cast<const uint4*>(grow + col);
-        __nv_bfloat162* g2 = reinterpret_cast<__nv_bfloat162*>(&gr);
+      for (int i = 0; i < 4; ++i) {
+        uint4 g = gr[c / 8 + i];
+        __nv_bfloat162* g2 = reinterpret_cast<__nv_bfloat162*>(&g);
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
-          const float a = ov[c8 + 2 * e] * inv / (1.f + __expf(-__bfloat162float(g2[e].x)));
-          const float b = ov[c8 + 2 * e + 1] * inv / (1.f + __expf(-__bfloat162float(g2[e].y)));
+          const float a = ov[8 * i + 2 * e] * inv *
+                          __fdividef(1.f, 1.f + __expf(-__bfloat162float(g2[e].x)));
+          const float b = ov[8 * i + 2 * e + 1] * inv *
+                          __fdividef(1.f, 1.f + __expf(-__bfloat162float(g2[e].y)));
           g2[e] = __floats2bfloat162_rn(a, b);
         }
-        *reinterpret_cast<uint4*>(grow + col) = gr;
+        if (store && c + i * 8 < n_col) *reinterpret_cast<uint4*>(grow + c + i * 8) = g;
       }
     }
     tc_fence_before();

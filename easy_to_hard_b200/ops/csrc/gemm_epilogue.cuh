@@ -83,34 +83,15 @@ __device__ __forceinline__ void epilogue8(const E2hGemmParams& p, int f, int t0,
       }
     } break;
     case E2H_EPI_RESIDUAL_F32: {
+      // the residual is updated in place: a reduction in L2 needs no round trip for the old value
+      // (one add per element and launch, so the sum is the same as load, add, store)
       float* out = static_cast<float*>(p.out);
-      const float* res = static_cast<const float*>(p.aux);
       if (!f_ok) break;
-      // loads first: `out` may alias `res`
-      float r[8];
-#pragma unroll
-      for (int j = 0; j < 8; ++j) r[j] = t0 + j < t_end ? res[(long long)(t0 + j) * p.ldo + f] : 0.f;
 #pragma unroll
       for (int j = 0; j < 8; ++j)
-        if (t0 + j < t_end) out[(long long)(t0 + j) * p.ldo + f] = r[j] + v[j];
-    } break;
-    case E2H_EPI_RESIDUAL: {
-      __nv_bfloat16* out = static_cast<__nv_bfloat16*>(p.out);
-      const __nv_bfloat16* res = static_cast<const __nv_bfloat16*>(p.aux);
-      // all residual loads first: `out` may alias `res`, so a load placed after a store could
-      // not be moved above it and the eight round trips would run one after another
-      float r[8];
-#pragma unroll
-      for (int j = 0; j < 8; ++j) {
-        const int t = t0 + j;
-        r[j] = (f_ok && t < t_end) ? __bfloat162float(res[(long long)t * p.ldo + f]) : 0.f;
-      }
-#pragma unroll
-      for (int j = 0; j < 8; ++j) {
-        const int t = t0 + j;
-        if (f_ok && t < t_end)
-          out[(long long)t * p.ldo + f] = __float2bfloat16_rn(bf16_round(v[j]) + r[j]);
-      }
+        if (t0 + j < t_end)
+          asm volatile("red.relaxed.gpu.global.add.f32 [%0], %1;" ::"l"(
+                           out + (long long)(t0 + j) * p.ldo + f), "f"(v[j]) : "memory");
     } break;
     case E2H_EPI_SWIGLU: {
       if constexpr (DUAL) {

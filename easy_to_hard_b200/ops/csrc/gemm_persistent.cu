@@ -641,6 +641,7 @@ extern "C" int e2h_gemm_persistent(const E2hGemmParams* pp, void* stream_v) {
   cudaStream_t stream = static_cast<cudaStream_t>(stream_v);
   if (p.F <= 0 || p.T <= 0 || p.K <= 0) return -1;
   if (p.splitk > 1 || p.a_tiled || p.n_groups > 0 || p.tail_from) return -3;
+  if (p.epi == E2H_EPI_RESIDUAL_F32 && p.aux != p.out) return -5;
   if (p.scale && (p.bias || p.act)) return -3;
   if ((p.bias || p.act) && p.epi != E2H_EPI_STORE_BF16 && p.epi != E2H_EPI_STORE_F32) return -3;
   if (p.dual && (p.a_mn_major || p.a2 == nullptr)) return -5;

@@ -591,6 +591,7 @@ extern "C" int e2h_gemm_umma(const E2hGemmParams* pp, void* stream_v) {
     return -5;
   if ((p.bias || p.act || p.tail_from) && p.epi != E2H_EPI_STORE_BF16 && p.epi != E2H_EPI_STORE_F32)
     return -5;
+  if (p.epi == E2H_EPI_RESIDUAL_F32 && p.aux != p.out) return -5;
   if (p.tail_from && (p.epi != E2H_EPI_STORE_BF16 || p.tail == nullptr)) return -5;
   const long long a_rows = (long long)p.F * (p.n_groups > 0 ? p.n_groups : 1);
   if ((p.lda % 8) || (p.ldb % 8) || (p.dual && (p.lda2 % 8))) return -6;  // 16-byte strides for TMA

@@ -17,7 +17,7 @@ enum E2hEpilogue : int {
   E2H_EPI_ROWMAJOR_F32_ACC = 5,  // out[f*ldo + t] (+)= acc  (fp32, weight gradients)
   E2H_EPI_ROWMAJOR_BF16 = 6,     // out[f*ldo + t] = bf16(acc)
   E2H_EPI_DUAL_STORE = 7,   // dual A: out[t*ldo+f] = bf16(acc1), out2[t*ldo2+f] = bf16(acc2)
-  E2H_EPI_RESIDUAL_F32 = 8, // out[t*ldo + f] = aux[t*ldo + f] + acc       (fp32 residual stream)
+  E2H_EPI_RESIDUAL_F32 = 8, // out[t*ldo + f] += acc, aux == out           (fp32 residual stream)
 };
 
 struct E2hGemmParams {

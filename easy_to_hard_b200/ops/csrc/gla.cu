@@ -264,6 +264,26 @@ __global__ void __launch_bounds__(256) gla_out_kernel(const E2hGlaParams p) {
   const float* o = p.o + w * p.vdim;
   T* g = static_cast<T*>(p.act) + t * p.ld + p.off_g + (long long)head * p.vdim;
   float ss = 0.f;
+  if ((p.vdim & 3) == 0 && (p.ld & 3) == 0 && (p.off_g & 3) == 0) {   // 4 columns per access
+    for (int i = lane * 4; i < p.vdim; i += 128) {
+      float x[4];
+      load4(o + i, x);
+      ss += x[0] * x[0] + x[1] * x[1] + x[2] * x[2] + x[3] * x[3];
+    }
+#pragma unroll
+    for (int m = 16; m > 0; m >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, m);
+    const float rstd = 1.f / sqrtf(ss / p.vdim + p.eps);
+    for (int i = lane * 4; i < p.vdim; i += 128) {
+      float x[4], z[4], w[4];
+      load4(o + i, x);
+      load4(g + i, z);
+      load4(p.norm + i, w);
+#pragma unroll
+      for (int e = 0; e < 4; ++e) x[e] = x[e] * rstd * w[e] * (z[e] * sigmoid_f(z[e]));
+      store4(g + i, x);
+    }
+    return;
+  }
   for (int i = lane; i < p.vdim; i += 32) ss += o[i] * o[i];
 #pragma unroll
   for (int m = 16; m > 0; m >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, m);

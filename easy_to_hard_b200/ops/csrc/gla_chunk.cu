@@ -38,13 +38,17 @@
 namespace e2h {
 
 constexpr int kC = 64;                 // tokens per chunk
-constexpr float kSteep = 40.f;         // decay over 16 tokens (in e) up to which e^{+} is harmless
+constexpr float kSteep = 40.f;         // decay (in e) up to which its inverse is harmless
 
 __device__ __forceinline__ int chunk_place(const E2hGlaParams& p, int sg, int c) {
   return p.seg[sg] / kC + sg + c;
 }
+// log sigmoid(z) to about 1e-7 absolute: it is only ever added up and exponentiated
 __device__ __forceinline__ float log_sigmoid_c(float z) {
-  return fminf(z, 0.f) - log1pf(expf(-fabsf(z)));
+  const float e = __expf(-fabsf(z));
+  // log(1 + e): Taylor series where 1 + e would round e away
+  const float l = e < 0.03f ? e * (1.f - e * (0.5f - e * (1.f / 3.f - e * 0.25f))) : __logf(1.f + e);
+  return fminf(z, 0.f) - l;
 }
 __device__ __forceinline__ void split_bf16(float x, float& hi, float& lo) {
   hi = bf16_round(x);
@@ -63,20 +67,34 @@ __device__ __forceinline__ void mma_16816(float* c, const uint32_t* a, const uin
 }
 
 constexpr int kPrepThreads = 256;
+constexpr int kAT = kC + 4;            // row pitch of the transposed decay input
 
 __host__ __device__ inline int prep_smem_bytes(int dim, int r) {
-  // b [64][dim + 4] fp32, q / k [64][dim + 8] bf16, a [64][r] fp32, partial sums [256]
-  return kC * (dim + 4) * 4 + 2 * kC * (dim + 8) * 2 + kC * r * 4 + kPrepThreads * 4;
+  // b [64][dim + 4] fp32, four bf16 [64][dim + 8] (q and k in two parts), a^T [r][68] fp32,
+  // partial sums [256]
+  return kC * (dim + 4) * 4 + 4 * kC * (dim + 8) * 2 + r * kAT * 4 + kPrepThreads * 4;
 }
 
-__global__ void __launch_bounds__(kPrepThreads) gla_chunk_prep_kernel(const E2hGlaParams p) {
+// 16 x 16 blocks (row, column) of A by warp; those above the diagonal are zero
+__constant__ unsigned char kPrepBlocks[8][2] = {{0x30, 0x31}, {0x32, 0x33}, {0x20, 0x21},
+                                                {0x22, 0x01}, {0x10, 0x11}, {0x00, 0x02},
+                                                {0x03, 0x12}, {0x13, 0x23}};
+
+// MMA fragments of rows r0.. and columns k0.. of a [64][pitch] bf16 tile
+__device__ __forceinline__ uint32_t frag(const __nv_bfloat16* x, int row, int col, int pitch) {
+  return *reinterpret_cast<const uint32_t*>(x + row * pitch + col);
+}
+
+__global__ void __launch_bounds__(kPrepThreads, 2) gla_chunk_prep_kernel(const E2hGlaParams p) {
   extern __shared__ __align__(16) uint8_t prep_raw[];
   const int D = p.dim, LB = D + 4, LQ = D + 8;
-  float* b_s = reinterpret_cast<float*>(prep_raw);                       // [64][LB]
-  __nv_bfloat16* q_s = reinterpret_cast<__nv_bfloat16*>(b_s + kC * LB);  // [64][LQ]
-  __nv_bfloat16* k_s = q_s + kC * LQ;
-  float* a_s = reinterpret_cast<float*>(k_s + kC * LQ);                  // [64][r]
-  float* sum_s = a_s + kC * p.r;                                         // [256]
+  float* b_s = reinterpret_cast<float*>(prep_raw);                        // [64][LB]
+  __nv_bfloat16* qh_s = reinterpret_cast<__nv_bfloat16*>(b_s + kC * LB);  // [64][LQ] each
+  __nv_bfloat16* ql_s = qh_s + kC * LQ;
+  __nv_bfloat16* kh_s = ql_s + kC * LQ;
+  __nv_bfloat16* kl_s = kh_s + kC * LQ;
+  float* at_s = reinterpret_cast<float*>(kl_s + kC * LQ);                 // [r][kAT]
+  float* sum_s = at_s + p.r * kAT;                                        // [256]
   pdl_launch_dependents();
   pdl_wait_prior();
   const int c = blockIdx.x, head = blockIdx.y, sg = blockIdx.z;
@@ -90,162 +108,193 @@ __global__ void __launch_bounds__(kPrepThreads) gla_chunk_prep_kernel(const E2hG
     return;
   }
   const int tid = threadIdx.x;
-  const __nv_bfloat16* act = static_cast<const __nv_bfloat16*>(p.act) + (long long)t0 * p.ld +
-                             (long long)head * D;
-  for (int i = tid; i < kC * (D / 8); i += kPrepThreads) {
-    const int t = i / (D / 8), d = (i - t * (D / 8)) * 8;
-    uint4 q = make_uint4(0, 0, 0, 0), k = q;
-    if (t < nt) {
-      q = *reinterpret_cast<const uint4*>(act + (long long)t * p.ld + p.off_q + d);
-      k = *reinterpret_cast<const uint4*>(act + (long long)t * p.ld + p.off_k + d);
-    }
-    *reinterpret_cast<uint4*>(q_s + t * LQ + d) = q;
-    *reinterpret_cast<uint4*>(k_s + t * LQ + d) = k;
+  for (int i = tid; i < kC * p.r; i += kPrepThreads) {
+    const int t = i / p.r, k = i - t * p.r;
+    at_s[k * kAT + t] = t < nt ? p.a[(long long)(t0 + t) * p.lda + k] : 0.f;
   }
-  for (int i = tid; i < nt * p.r; i += kPrepThreads)
-    a_s[i] = p.a[(long long)(t0 + i / p.r) * p.lda + i % p.r];
   __syncthreads();
   // running sums of log alpha: `ng` groups of threads take consecutive runs of tokens of a column
-  const int ng = kPrepThreads / D, run = (kC + ng - 1) / ng;
   {
-    const int g = tid / D, d = tid - g * D;
-    float acc = 0.f;
-    if (g < ng) {
+    const int ng = min(kPrepThreads / D, 16), run = ((kC + ng - 1) / ng + 3) / 4 * 4;   // <= 32
+    const int g = tid / D, d = tid - g * D, tb = g * run;
+    const bool work = g < ng && tb < kC;
+    float z[32];
+    float add = 0.f;
+    if (work) {
       const __nv_bfloat16* w = static_cast<const __nv_bfloat16*>(p.w2) +
                                ((long long)head * D + d) * p.ldw;
+      const bool wvec = (p.ldw & 7) == 0 && (p.r & 7) == 0 &&
+                        (reinterpret_cast<uintptr_t>(p.w2) & 15) == 0;
       const float bias = p.b2[head * D + d];
-      for (int t = g * run; t < min(kC, (g + 1) * run); ++t) {
-        if (t < nt) {
-          float z = bias;
-          for (int i = 0; i < p.r; ++i) z = fmaf(to_f(w[i]), a_s[t * p.r + i], z);
-          acc += log_sigmoid_c(z) * p.inv_tau;
+#pragma unroll
+      for (int j = 0; j < 32; ++j) z[j] = bias;
+      for (int i0 = 0; i0 < p.r; i0 += 8) {
+        float wv[8];
+        if (wvec) {
+          load8(w + i0, wv);
+        } else {
+#pragma unroll
+          for (int e = 0; e < 8; ++e) wv[e] = i0 + e < p.r ? to_f(w[i0 + e]) : 0.f;
         }
-        b_s[t * LB + d] = acc;
+#pragma unroll
+        for (int e = 0; e < 8; ++e) {
+          if (i0 + e >= p.r) break;
+          const float* at = at_s + (i0 + e) * kAT + tb;
+#pragma unroll
+          for (int j = 0; j < 8; ++j) {
+            if (4 * j >= run) break;
+            const float4 av = *reinterpret_cast<const float4*>(at + 4 * j);
+            z[4 * j] = fmaf(wv[e], av.x, z[4 * j]);
+            z[4 * j + 1] = fmaf(wv[e], av.y, z[4 * j + 1]);
+            z[4 * j + 2] = fmaf(wv[e], av.z, z[4 * j + 2]);
+            z[4 * j + 3] = fmaf(wv[e], av.w, z[4 * j + 3]);
+          }
+        }
+      }
+      float acc = 0.f;
+#pragma unroll
+      for (int j = 0; j < 32; ++j) {
+        if (j < run && tb + j < nt) acc += log_sigmoid_c(z[j]) * p.inv_tau;
+        z[j] = acc;
       }
       sum_s[tid] = acc;
     }
     __syncthreads();
-    if (g < ng && g > 0) {
-      float add = 0.f;
+    if (work) {
       for (int k = 0; k < g; ++k) add += sum_s[k * D + d];
-      for (int t = g * run; t < min(kC, (g + 1) * run); ++t) b_s[t * LB + d] += add;
+#pragma unroll
+      for (int j = 0; j < 32; ++j)
+        if (j < run && tb + j < kC) b_s[(tb + j) * LB + d] = z[j] + add;
     }
   }
   __syncthreads();
-  // decayed q and k, in two parts each
+  const float* b_end = b_s + (kC - 1) * LB;
+  bool mine = false;
+  for (int d = tid; d < D; d += kPrepThreads) {
+    mine = mine || !(-b_end[d] <= kSteep);
+    p.cg[((long long)place * p.H + head) * D + d] = __expf(b_end[d]);
+  }
+  // steep: the inverse decay of the chunk leaves the fp32 range; A then takes its exact form and
+  // the shared tiles hold the plain q and k
+  const bool steep = __syncthreads_or(mine) != 0;
+  const __nv_bfloat16* act = static_cast<const __nv_bfloat16*>(p.act) + (long long)t0 * p.ld +
+                             (long long)head * D;
   const long long row0 = ((long long)place * p.H + head) * kC;
   const long long part = (long long)p.chunks * p.H * kC * D;
   __nv_bfloat16* cq = static_cast<__nv_bfloat16*>(p.cq) + row0 * D;
   __nv_bfloat16* ck = static_cast<__nv_bfloat16*>(p.ck) + row0 * D;
   for (int i = tid; i < kC * (D / 8); i += kPrepThreads) {
     const int t = i / (D / 8), d = (i - t * (D / 8)) * 8;
-    float q[8], k[8];
-    load8(q_s + t * LQ + d, q);
-    load8(k_s + t * LQ + d, k);
-    uint32_t qh[4], ql[4], kh[4], kl[4];
+    float q[8], k[8], b[8];
+    if (t < nt) {
+      load8(act + (long long)t * p.ld + p.off_q + d, q);
+      load8(act + (long long)t * p.ld + p.off_k + d, k);
+    } else {
+#pragma unroll
+      for (int e = 0; e < 8; ++e) q[e] = k[e] = 0.f;
+    }
+    load8(b_s + t * LB + d, b);
+    uint32_t qh[4], ql[4], kh[4], kl[4], eh[4], el[4];
 #pragma unroll
     for (int e = 0; e < 8; e += 2) {
-      float h0, l0, h1, l1;
-      const float b0 = b_s[t * LB + d + e], b1 = b_s[t * LB + d + e + 1];
-      split_bf16(q[e] * p.qscale * expf(b0), h0, l0);
-      split_bf16(q[e + 1] * p.qscale * expf(b1), h1, l1);
-      qh[e / 2] = pack2(h0, h1);
-      ql[e / 2] = pack2(l0, l1);
-      split_bf16(k[e] * expf(b_s[(kC - 1) * LB + d + e] - b0), h0, l0);
-      split_bf16(k[e + 1] * expf(b_s[(kC - 1) * LB + d + e + 1] - b1), h1, l1);
-      kh[e / 2] = pack2(h0, h1);
-      kl[e / 2] = pack2(l0, l1);
+      float h[2], l[2], ih[2], il[2], xh[2], xl[2];
+#pragma unroll
+      for (int u = 0; u < 2; ++u) {
+        const float eb = __expf(b[e + u]);
+        split_bf16(q[e + u] * p.qscale * eb, h[u], l[u]);
+        if (!steep) {
+          const float ki = __fdividef(k[e + u], eb);
+          split_bf16(ki, ih[u], il[u]);
+          split_bf16(ki * __expf(b_end[d + e + u]), xh[u], xl[u]);
+        } else {
+          split_bf16(k[e + u] * __expf(b_end[d + e + u] - b[e + u]), xh[u], xl[u]);
+        }
+      }
+      qh[e / 2] = pack2(h[0], h[1]);
+      ql[e / 2] = pack2(l[0], l[1]);
+      eh[e / 2] = pack2(xh[0], xh[1]);
+      el[e / 2] = pack2(xl[0], xl[1]);
+      if (!steep) {
+        kh[e / 2] = pack2(ih[0], ih[1]);
+        kl[e / 2] = pack2(il[0], il[1]);
+      }
     }
     const long long o = (long long)t * D + d;
-    *reinterpret_cast<uint4*>(cq + o) = make_uint4(qh[0], qh[1], qh[2], qh[3]);
-    *reinterpret_cast<uint4*>(cq + part + o) = make_uint4(ql[0], ql[1], ql[2], ql[3]);
-    *reinterpret_cast<uint4*>(ck + o) = make_uint4(kh[0], kh[1], kh[2], kh[3]);
-    *reinterpret_cast<uint4*>(ck + part + o) = make_uint4(kl[0], kl[1], kl[2], kl[3]);
+    const uint4 qh4 = make_uint4(qh[0], qh[1], qh[2], qh[3]);
+    const uint4 ql4 = make_uint4(ql[0], ql[1], ql[2], ql[3]);
+    *reinterpret_cast<uint4*>(cq + o) = qh4;
+    *reinterpret_cast<uint4*>(cq + part + o) = ql4;
+    *reinterpret_cast<uint4*>(ck + o) = make_uint4(eh[0], eh[1], eh[2], eh[3]);
+    *reinterpret_cast<uint4*>(ck + part + o) = make_uint4(el[0], el[1], el[2], el[3]);
+    if (!steep) {
+      *reinterpret_cast<uint4*>(qh_s + t * LQ + d) = qh4;
+      *reinterpret_cast<uint4*>(ql_s + t * LQ + d) = ql4;
+      *reinterpret_cast<uint4*>(kh_s + t * LQ + d) = make_uint4(kh[0], kh[1], kh[2], kh[3]);
+      *reinterpret_cast<uint4*>(kl_s + t * LQ + d) = make_uint4(kl[0], kl[1], kl[2], kl[3]);
+    } else {
+      store4(qh_s + t * LQ + d, q);
+      store4(qh_s + t * LQ + d + 4, q + 4);
+      store4(kh_s + t * LQ + d, k);
+      store4(kh_s + t * LQ + d + 4, k + 4);
+    }
   }
-  for (int d = tid; d < D; d += kPrepThreads)
-    p.cg[((long long)place * p.H + head) * D + d] = expf(b_s[(kC - 1) * LB + d]);
-  // A in 16 x 16 blocks: 10 on or below the diagonal, 6 above it that are zero
+  __syncthreads();
+  // A in 16 x 16 blocks
   const int warp = tid >> 5, lane = tid & 31;
-  const int gq = lane >> 2, cq2 = (lane & 3) * 2;
+  const int gr = lane >> 2, c2 = (lane & 3) * 2;
   __nv_bfloat16* ca = static_cast<__nv_bfloat16*>(p.ca) + row0 * kC;
   const long long apart = (long long)p.chunks * p.H * kC * kC;
-  for (int blk = warp; blk < 16; blk += kPrepThreads / 32) {
-    const int bi = blk >> 2, bj = blk & 3;         // token rows 16 bi.., source columns 16 bj..
+  for (int n = 0; n < 2; ++n) {
+    const int bi = kPrepBlocks[warp][n] >> 4, bj = kPrepBlocks[warp][n] & 15;
     float acc[2][4];
 #pragma unroll
     for (int x = 0; x < 2; ++x)
 #pragma unroll
       for (int y = 0; y < 4; ++y) acc[x][y] = 0.f;
-    if (bj <= bi) {
-      // reference sum: that before the block's first token row
-      const float* ref = bi > 0 ? b_s + (16 * bi - 1) * LB : nullptr;
-      bool steep = false;
-      if (bj == bi) {
-        float mx = 0.f;
-        for (int d = lane; d < D; d += 32)
-          mx = fmaxf(mx, (ref ? ref[d] : 0.f) - b_s[(16 * bi + 15) * LB + d]);
-        steep = __any_sync(0xffffffffu, !(mx <= kSteep));
-      }
-      if (!steep) {
-        const int ra = 16 * bi + gq, rb = 16 * bj + gq;
-        for (int k0 = 0; k0 < D; k0 += 16) {
-          uint32_t ah[4], al[4], bh[2][2], bl[2][2];
+    if (bj <= bi && !steep) {
+      const int ra = 16 * bi + gr, rb = 16 * bj + gr;
+      for (int k0 = 0; k0 < D; k0 += 16) {
+        uint32_t ah[4], al[4];
 #pragma unroll
-          for (int x = 0; x < 4; ++x) {            // (row, k): (g, c) (g + 8, c) (g, c + 8) ..
-            const int t = ra + (x & 1) * 8, d = k0 + cq2 + (x >> 1) * 8;
-            float h[2], l[2];
-#pragma unroll
-            for (int e = 0; e < 2; ++e)
-              split_bf16(to_f(q_s[t * LQ + d + e]) * p.qscale *
-                             expf(b_s[t * LB + d + e] - (ref ? ref[d + e] : 0.f)), h[e], l[e]);
-            ah[x] = pack2(h[0], h[1]);
-            al[x] = pack2(l[0], l[1]);
-          }
-#pragma unroll
-          for (int nb = 0; nb < 2; ++nb)
-#pragma unroll
-            for (int x = 0; x < 2; ++x) {
-              const int s = rb + nb * 8, d = k0 + cq2 + x * 8;
-              float h[2], l[2];
-#pragma unroll
-              for (int e = 0; e < 2; ++e)
-                split_bf16(to_f(k_s[s * LQ + d + e]) *
-                               expf((ref ? ref[d + e] : 0.f) - b_s[s * LB + d + e]), h[e], l[e]);
-              bh[nb][x] = pack2(h[0], h[1]);
-              bl[nb][x] = pack2(l[0], l[1]);
-            }
-#pragma unroll
-          for (int nb = 0; nb < 2; ++nb) {
-            mma_16816(acc[nb], ah, bh[nb]);
-            mma_16816(acc[nb], ah, bl[nb]);
-            mma_16816(acc[nb], al, bh[nb]);
-          }
+        for (int x = 0; x < 4; ++x) {              // (row, k): (g, c) (g + 8, c) (g, c + 8) ..
+          ah[x] = frag(qh_s, ra + (x & 1) * 8, k0 + c2 + (x >> 1) * 8, LQ);
+          al[x] = frag(ql_s, ra + (x & 1) * 8, k0 + c2 + (x >> 1) * 8, LQ);
         }
-      } else {
 #pragma unroll
-        for (int nb = 0; nb < 2; ++nb)
+        for (int nb = 0; nb < 2; ++nb) {
+          uint32_t bh[2], bl[2];
 #pragma unroll
-          for (int y = 0; y < 4; ++y) {
-            const int t = 16 * bi + gq + (y >> 1) * 8, s = 16 * bj + nb * 8 + cq2 + (y & 1);
-            if (s > t) continue;
-            float v = 0.f;
-            for (int d = 0; d < D; ++d)
-              v = fmaf(to_f(q_s[t * LQ + d]) * p.qscale,
-                       to_f(k_s[s * LQ + d]) * expf(b_s[t * LB + d] - b_s[s * LB + d]), v);
-            acc[nb][y] = v;
+          for (int x = 0; x < 2; ++x) {
+            bh[x] = frag(kh_s, rb + nb * 8, k0 + c2 + x * 8, LQ);
+            bl[x] = frag(kl_s, rb + nb * 8, k0 + c2 + x * 8, LQ);
           }
+          mma_16816(acc[nb], ah, bh);
+          mma_16816(acc[nb], ah, bl);
+          mma_16816(acc[nb], al, bh);
+        }
       }
+    } else if (bj <= bi) {
+#pragma unroll
+      for (int nb = 0; nb < 2; ++nb)
+#pragma unroll
+        for (int y = 0; y < 4; ++y) {
+          const int t = 16 * bi + gr + (y >> 1) * 8, s = 16 * bj + nb * 8 + c2 + (y & 1);
+          if (s > t) continue;
+          float v = 0.f;
+          for (int d = 0; d < D; ++d)
+            v = fmaf(to_f(qh_s[t * LQ + d]) * p.qscale,
+                     to_f(kh_s[s * LQ + d]) * __expf(b_s[t * LB + d] - b_s[s * LB + d]), v);
+          acc[nb][y] = v;
+        }
     }
 #pragma unroll
     for (int nb = 0; nb < 2; ++nb)
 #pragma unroll
-      for (int half = 0; half < 2; ++half) {
-        const int t = 16 * bi + gq + half * 8, s = 16 * bj + nb * 8 + cq2;
-        const float x = s <= t ? acc[nb][2 * half] : 0.f;
-        const float y = s + 1 <= t ? acc[nb][2 * half + 1] : 0.f;
+      for (int hf = 0; hf < 2; ++hf) {
+        const int t = 16 * bi + gr + hf * 8, s = 16 * bj + nb * 8 + c2;
         float h0, l0, h1, l1;
-        split_bf16(x, h0, l0);
-        split_bf16(y, h1, l1);
+        split_bf16(s <= t ? acc[nb][2 * hf] : 0.f, h0, l0);
+        split_bf16(s + 1 <= t ? acc[nb][2 * hf + 1] : 0.f, h1, l1);
         *reinterpret_cast<uint32_t*>(ca + t * kC + s) = pack2(h0, h1);
         *reinterpret_cast<uint32_t*>(ca + apart + t * kC + s) = pack2(l0, l1);
       }
@@ -570,7 +619,7 @@ extern "C" int e2h_gla_chunk(const E2hGlaParams* pp, void* stream_v) {
   if (!p.o || !p.cg || !p.state || !p.status || p.chunks < p.n / kC + p.n_seg) return -3;
   if (2LL * p.chunks * p.H * kC > 0x7fffffffLL) return -4;
   const int smem = prep_smem_bytes(p.dim, p.r);
-  if (smem > 200 * 1024) return -5;
+  if (smem > 200 * 1024 || p.r > 128) return -5;
   static std::once_flag once;
   static cudaError_t err = cudaSuccess;
   std::call_once(once, [] {

@@ -71,22 +71,30 @@ __device__ __forceinline__ void copy_row(T* dst, const T* src, int W) {
   }
 }
 
+constexpr int kRouteThreads = 512;
+constexpr int kRouteLogits = 8192;   // logits staged in shared memory
+
 template <typename T>
-__global__ void __launch_bounds__(256)
+__global__ void __launch_bounds__(kRouteThreads)
 moe_route_small_kernel(const float* z, long long ldz, int n, int E, int top, const T* h,
                        long long ldh, int W, T* hg, long long ldg, int* off, int* place, float* w) {
   __shared__ int sel[kMoeSmall];
   __shared__ int count[kMoeMaxExperts];
   __shared__ int my_off[kMoeMaxTop], my_before[kMoeMaxTop];
+  extern __shared__ float z_s[];
   pdl_launch_dependents();
   pdl_wait_prior();
+  const bool staged = n * E <= kRouteLogits;
+  if (staged)
+    for (int i = threadIdx.x; i < n * E; i += blockDim.x) z_s[i] = z[i / E * ldz + i % E];
   const int t_me = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   for (int e = threadIdx.x; e < E; e += blockDim.x) count[e] = 0;
   if (threadIdx.x < top) my_off[threadIdx.x] = my_before[threadIdx.x] = 0;
+  __syncthreads();
   for (int t = warp; t < n; t += blockDim.x >> 5) {
     int idx[kMoeMaxTop];
     float val[kMoeMaxTop];
-    warp_topk(z + t * ldz, E, top, idx, val);
+    warp_topk(staged ? z_s + t * E : z + t * ldz, E, top, idx, val);
     if (lane == 0) {
       for (int j = 0; j < top; ++j) {
         sel[t * top + j] = idx[j];
@@ -207,7 +215,8 @@ static int route(const float* z, long long ldz, int n, int E, int top, const voi
                  int W, void* hg, long long ldg, int* off, int* place, float* w, int* sel,
                  cudaStream_t s) {
   if (n * top <= kMoeSmall && n <= 256)
-    return (int)launch(moe_route_small_kernel<T>, dim3(n), dim3(256), 0, s, z, ldz, n, E, top,
+    return (int)launch(moe_route_small_kernel<T>, dim3(n), dim3(kRouteThreads),
+                       n * E <= kRouteLogits ? (size_t)n * E * 4 : 0, s, z, ldz, n, E, top,
                        static_cast<const T*>(h), ldh, W, static_cast<T*>(hg), ldg, off, place, w);
   int r = (int)launch(moe_topk_kernel, dim3((n + 7) / 8), dim3(256), 0, s, z, ldz, n, E, top, sel, w);
   if (r) return r;
