@@ -16,8 +16,8 @@
 //                of the cluster and merged through distributed shared memory. In its fused form
 //                (decode) it does the work of attn_prep itself, so that a decode step has one
 //                attention kernel; otherwise every token, also of a prompt, reads its keys from
-//                the cache. This kernel is the fp32 path and the path of head sizes and portions
-//                that the tensor-core prompt kernel does not take.
+//                the cache (portions and head sizes that the tensor-core prompt kernel does not
+//                take). Two forms: fp32 on the CUDA cores, bf16 on warp-level matrix products.
 #include <cooperative_groups.h>
 #include <cuda_bf16.h>
 #include <cuda_runtime.h>
@@ -245,6 +245,58 @@ __global__ void __launch_bounds__(256) attn_prep_kernel(const AttnWindowParams p
 constexpr int kWinThreads = 128;
 constexpr int kWinUnroll = 4;      // keys a lane group has in flight
 
+// Merges the (m, l, acc) of a CTA's key groups (in shared memory), then those of the cluster's CTAs,
+// and writes the gated heads: every CTA of the cluster finishes its share of the columns.
+template <typename T, int GROUPS, int R, int DP>
+__device__ __forceinline__ void window_finish(const AttnWindowParams& p,
+                                              cg::cluster_group& cluster, const float* mrg,
+                                              float* acc_s, float (*fin)[2], T* row, int h0,
+                                              int nr, int rank) {
+  __syncthreads();
+  for (int i = threadIdx.x; i < R * DP; i += kWinThreads) {
+    const int r = i / DP, d = i - r * DP;
+    float mx = -FLT_MAX;
+    for (int k = 0; k < GROUPS; ++k) mx = fmaxf(mx, mrg[(k * R + r) * 2]);
+    float a = 0.f, ls = 0.f;
+    for (int k = 0; k < GROUPS; ++k) {
+      const float w = exp2f(mrg[(k * R + r) * 2] - mx);
+      a += w * acc_s[(k * R + r) * DP + d];
+      ls += w * mrg[(k * R + r) * 2 + 1];
+    }
+    acc_s[i] = a;                       // entry (0, r, d) is read by this thread only
+    if (d == 0) {
+      fin[r][0] = mx;
+      fin[r][1] = ls;
+    }
+  }
+  if (p.splits > 1) cluster.sync();
+  else __syncthreads();
+  // merge the cluster: every CTA finishes its share of the columns
+  const int total = nr * p.vdim;
+  const int per = (total + p.splits - 1) / p.splits;
+  for (int i = rank * per + threadIdx.x; i < min(total, (rank + 1) * per); i += kWinThreads) {
+    const int r = i / p.vdim, d = i - r * p.vdim;
+    float o;
+    if (p.splits > 1) {
+      float mx = -FLT_MAX;
+      for (int k = 0; k < p.splits; ++k) mx = fmaxf(mx, cluster.map_shared_rank(&fin[r][0], k)[0]);
+      float a = 0.f, ls = 0.f;
+      for (int k = 0; k < p.splits; ++k) {
+        const float* f = cluster.map_shared_rank(&fin[r][0], k);
+        const float w = exp2f(f[0] - mx);
+        ls += w * f[1];
+        a += w * cluster.map_shared_rank(acc_s, k)[r * DP + d];
+      }
+      o = a / ls;
+    } else {
+      o = acc_s[r * DP + d] / fin[r][1];
+    }
+    T* gate = row + p.off_g + (h0 + r) * p.vdim + d;
+    *gate = from_f<T>(o * sigmoid_f(to_f(*gate)));
+  }
+  if (p.splits > 1) cluster.sync();     // peers may still read this CTA's shared memory
+}
+
 // LPK lanes share a key (8 elements each), R query heads of the kv head's group per CTA.
 template <typename T, int LPK, int R, bool FUSED>
 __global__ void __launch_bounds__(kWinThreads) attn_window_kernel(const AttnWindowParams p) {
@@ -414,59 +466,242 @@ __global__ void __launch_bounds__(kWinThreads) attn_window_kernel(const AttnWind
 #pragma unroll
     for (int e = 0; e < 8; ++e) acc_s[(grp * R + r) * LPK * 8 + gl * 8 + e] = acc[r][e];
   }
-  __syncthreads();
-  for (int i = threadIdx.x; i < R * LPK * 8; i += kWinThreads) {
-    const int r = i / (LPK * 8), d = i - r * (LPK * 8);
-    float mx = -FLT_MAX;
-    for (int k = 0; k < GROUPS; ++k) mx = fmaxf(mx, mrg[(k * R + r) * 2]);
-    float a = 0.f, ls = 0.f;
-    for (int k = 0; k < GROUPS; ++k) {
-      const float w = exp2f(mrg[(k * R + r) * 2] - mx);
-      a += w * acc_s[(k * R + r) * LPK * 8 + d];
-      ls += w * mrg[(k * R + r) * 2 + 1];
-    }
-    acc_s[i] = a;                       // entry (0, r, d) is read by this thread only
-    if (d == 0) {
-      fin[r][0] = mx;
-      fin[r][1] = ls;
-    }
-  }
-  if (p.splits > 1) cluster.sync();
-  else __syncthreads();
-  // merge the cluster: every CTA finishes its share of the columns
-  const int total = nr * p.vdim;
-  const int per = (total + p.splits - 1) / p.splits;
-  for (int i = rank * per + threadIdx.x; i < min(total, (rank + 1) * per); i += kWinThreads) {
-    const int r = i / p.vdim, d = i - r * p.vdim;
-    float o;
-    if (p.splits > 1) {
-      float mx = -FLT_MAX;
-      for (int k = 0; k < p.splits; ++k) mx = fmaxf(mx, cluster.map_shared_rank(&fin[r][0], k)[0]);
-      float a = 0.f, ls = 0.f;
-      for (int k = 0; k < p.splits; ++k) {
-        const float* f = cluster.map_shared_rank(&fin[r][0], k);
-        const float w = exp2f(f[0] - mx);
-        ls += w * f[1];
-        a += w * cluster.map_shared_rank(acc_s, k)[r * LPK * 8 + d];
-      }
-      o = a / ls;
-    } else {
-      o = acc_s[r * LPK * 8 + d] / fin[r][1];
-    }
-    T* gate = row + p.off_g + (h0 + r) * p.vdim + d;
-    *gate = from_f<T>(o * sigmoid_f(to_f(*gate)));
-  }
-  if (p.splits > 1) cluster.sync();     // peers may still read this CTA's shared memory
+  window_finish<T, GROUPS, R, LPK * 8>(p, cluster, mrg, acc_s, fin, row, h0, nr, rank);
 }
 
-template <typename T, int LPK, int R, bool FUSED>
-static int win_launch(const AttnWindowParams& p, cudaStream_t stream) {
-  constexpr int GROUPS = kWinThreads / LPK;
-  const size_t smem = sizeof(float) * (R * LPK * 8 + 2 * LPK * 8 + GROUPS * R * 2 +
-                                       (size_t)GROUPS * R * LPK * 8);
-  static_assert(sizeof(float) * (R * LPK * 8 + 2 * LPK * 8 + GROUPS * R * 2 +
-                                 GROUPS * R * LPK * 8) < 48 * 1024, "fits the default limit");
-  const int per_g = p.H / p.G, n_rb = (per_g + R - 1) / R;
+__device__ __forceinline__ void window_mma(float* c, uint32_t a0, uint32_t a2, uint32_t b0,
+                                           uint32_t b1) {
+  asm volatile(
+      "mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, "
+      "{%8,%9}, {%0,%1,%2,%3};"
+      : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
+      : "r"(a0), "r"(0u), "r"(a2), "r"(0u), "r"(b0), "r"(b1));
+}
+__device__ __forceinline__ uint32_t pack_bf16(float a, float b) {
+  const __nv_bfloat162 v = __floats2bfloat162_rn(a, b);
+  return *reinterpret_cast<const uint32_t*>(&v);
+}
+
+// bf16 form: the query heads of a group (up to 8) are the rows of warp-level matrix products, so a
+// key costs a few instructions however many heads share it and the kernel is a stream of the cache.
+// A warp takes 16 keys at a time. Lane (g, c) = (lane / 4, lane % 4). The contraction of q k^T runs
+// over the head columns in any order as long as both operands agree: the lane's 16-byte piece of key
+// g holds the fragment words of two k-steps. The scores leave in the layout of the A operand of
+// p v; the value fragments pair two keys, packed from the 16-byte pieces of both (the columns of the
+// result are permuted accordingly).
+template <int LPK, bool FUSED>
+__global__ void __launch_bounds__(kWinThreads) attn_window_mma_kernel(const AttnWindowParams p) {
+  using T = __nv_bfloat16;
+  constexpr int R = 8, DP = LPK * 8, GROUPS = kWinThreads / 32;
+  constexpr int KI = (LPK + 3) / 4;              // 16-byte pieces of a key per lane
+  constexpr int VI = (LPK + 7) / 8;              // value pieces of one key per lane
+  extern __shared__ __align__(16) float win_s[];
+  float* mrg = win_s;                            // [GROUPS][R] m, l
+  float* acc_s = mrg + GROUPS * R * 2;           // [GROUPS][R][DP]; group 0 = the CTA's sum
+  T* q_s = reinterpret_cast<T*>(acc_s + GROUPS * R * DP);   // [R][DP]
+  T* k_new = q_s + R * DP;                       // fused: the token's own key and value
+  T* v_new = k_new + DP;
+  __shared__ float red[33];
+  __shared__ float fin[R][2];
+
+  cg::cluster_group cluster = cg::this_cluster();
+  pdl_launch_dependents();
+  pdl_wait_prior();
+  const int rank = blockIdx.x, t = blockIdx.z;
+  const int per_g = p.H / p.G;
+  const int n_rb = (per_g + R - 1) / R;
+  const int g = blockIdx.y / n_rb, rb = blockIdx.y - g * n_rb;
+  const int h0 = g * per_g + rb * R;
+  const int nr = min(R, per_g - rb * R);
+  int pos = p.pos[t], slot = p.slot[t];
+  const bool ok = pos >= 0 && pos < p.smax && slot >= 0 && slot < p.slots;
+  if (!ok) {
+    if (threadIdx.x == 0) atomicCAS(p.status, 0, kStatusBadArgs);
+    pos = min(max(pos, 0), p.smax - 1);
+    slot = min(max(slot, 0), p.slots - 1);
+  }
+  T* row = static_cast<T*>(p.act) + t * p.ld;
+  const T* q = row + p.off_q;
+  const long long hb = (long long)slot * p.G + g;
+  T* kc = static_cast<T*>(p.kc) + hb * p.smax * p.dimp;
+  T* vc = static_cast<T*>(p.vc) + hb * p.smax * p.vdimp;
+  const float* cs = p.rot_table + (long long)pos * (p.rot & ~1);
+  const float sl2 = p.scale * 1.4426950408889634f;
+
+  float rq = 1.f, rk = 1.f;
+  if constexpr (FUSED) {
+    if (p.qn) rq = rms_of(q, p.H * p.dim, p.eps, red);
+    if (p.kn && rank == 0) rk = rms_of(row + p.off_k, p.G * p.dim, p.eps, red);
+  }
+  for (int i = threadIdx.x; i < R * DP; i += kWinThreads) {
+    const int r = i / DP, d = i - r * DP;
+    T x = from_f<T>(0.f);
+    if (r < nr && d < p.dim) {
+      const int h = h0 + r;
+      if constexpr (FUSED)
+        x = from_f<T>(norm_rot(q + h * p.dim, p.qn ? p.qn + h * p.dim : nullptr, rq, d, p.rot,
+                               cs));
+      else
+        x = q[h * p.dim + d];
+    }
+    q_s[i] = x;
+  }
+  if constexpr (FUSED) {
+    if (rank == 0) {
+      for (int d = threadIdx.x; d < DP; d += kWinThreads) {
+        T x = from_f<T>(0.f), y = x;
+        if (d < p.dim)
+          x = from_f<T>(norm_rot(row + p.off_k + g * p.dim, p.kn ? p.kn + g * p.dim : nullptr, rk,
+                                 d, p.rot, cs));
+        if (d < p.vdim) y = row[p.off_v + g * p.vdim + d];
+        if (rb == 0 && ok) {
+          if (d < p.dim) kc[(long long)pos * p.dimp + d] = x;
+          if (d < p.vdim) vc[(long long)pos * p.vdimp + d] = y;
+        }
+        k_new[d] = x;
+        v_new[d] = y;
+      }
+    }
+  }
+  __syncthreads();
+
+  const int last = FUSED ? pos : pos + 1;
+  int lo = p.window > 0 ? pos - p.window + 1 : 0;
+  lo = max(lo, 0);
+  const int n_keep = min(p.keep, lo);
+  const int n_keys = n_keep + max(last - lo, 0);
+  const int k_begin = (int)((long long)n_keys * rank / p.splits);
+  const int k_end = (int)((long long)n_keys * (rank + 1) / p.splits);
+
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int gr = lane >> 2, c = lane & 3;
+  const int k_pieces = p.dimp / 8, v_pieces = p.vdimp / 8;
+  uint32_t qa[KI][4];                            // fragment words of head gr, pieces c + 4 i
+#pragma unroll
+  for (int i = 0; i < KI; ++i) {
+    const uint4 x = *reinterpret_cast<const uint4*>(q_s + gr * DP + min(c + 4 * i, LPK - 1) * 8);
+    const bool in = c + 4 * i < LPK;
+    qa[i][0] = in ? x.x : 0;
+    qa[i][1] = in ? x.y : 0;
+    qa[i][2] = in ? x.z : 0;
+    qa[i][3] = in ? x.w : 0;
+  }
+  float acc[VI][8][4];
+#pragma unroll
+  for (int i = 0; i < VI; ++i)
+#pragma unroll
+    for (int j = 0; j < 8; ++j)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) acc[i][j][e] = 0.f;
+  float m = -FLT_MAX, l = 0.f;
+  const uint4 zero4 = make_uint4(0, 0, 0, 0);
+
+  // 16 keys: key(x), val(x) point at key x of them or are null
+  auto absorb = [&](auto key, auto val) {
+    uint4 kf[2][KI], vf[4][VI];
+#pragma unroll
+    for (int x = 0; x < 2; ++x) {
+      const T* kp = key(gr + 8 * x);
+#pragma unroll
+      for (int i = 0; i < KI; ++i)
+        kf[x][i] = kp && c + 4 * i < k_pieces
+                       ? *reinterpret_cast<const uint4*>(kp + (c + 4 * i) * 8) : zero4;
+    }
+#pragma unroll
+    for (int x = 0; x < 4; ++x) {
+      const T* vp = val(2 * c + (x & 1) + 8 * (x >> 1));
+#pragma unroll
+      for (int i = 0; i < VI; ++i)
+        vf[x][i] = vp && gr + 8 * i < v_pieces
+                       ? *reinterpret_cast<const uint4*>(vp + (gr + 8 * i) * 8) : zero4;
+    }
+    float s[2][4];
+#pragma unroll
+    for (int x = 0; x < 2; ++x) {
+#pragma unroll
+      for (int e = 0; e < 4; ++e) s[x][e] = 0.f;
+#pragma unroll
+      for (int i = 0; i < KI; ++i) {
+        window_mma(s[x], qa[i][0], qa[i][1], kf[x][i].x, kf[x][i].y);
+        window_mma(s[x], qa[i][2], qa[i][3], kf[x][i].z, kf[x][i].w);
+      }
+    }
+    // this lane: head gr, keys 2c, 2c + 1, 2c + 8, 2c + 9
+    float mx = m;
+#pragma unroll
+    for (int x = 0; x < 2; ++x)
+#pragma unroll
+      for (int e = 0; e < 2; ++e) {
+        s[x][e] = key(2 * c + e + 8 * x) ? s[x][e] * sl2 : -FLT_MAX;
+        mx = fmaxf(mx, s[x][e]);
+      }
+    mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 1));
+    mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 2));
+    const float al = exp2f(m - mx);
+    m = mx;
+    float w[2][2];
+    l *= al;
+#pragma unroll
+    for (int x = 0; x < 2; ++x)
+#pragma unroll
+      for (int e = 0; e < 2; ++e) {
+        w[x][e] = s[x][e] == -FLT_MAX ? 0.f : exp2f(s[x][e] - mx);
+        l += w[x][e];
+      }
+    const uint32_t pa0 = pack_bf16(w[0][0], w[0][1]), pa2 = pack_bf16(w[1][0], w[1][1]);
+#pragma unroll
+    for (int i = 0; i < VI; ++i) {
+      const uint32_t* v0 = reinterpret_cast<const uint32_t*>(&vf[0][i]);
+      const uint32_t* v1 = reinterpret_cast<const uint32_t*>(&vf[1][i]);
+      const uint32_t* v2 = reinterpret_cast<const uint32_t*>(&vf[2][i]);
+      const uint32_t* v3 = reinterpret_cast<const uint32_t*>(&vf[3][i]);
+#pragma unroll
+      for (int j = 0; j < 8; ++j) {
+        acc[i][j][0] *= al;
+        acc[i][j][1] *= al;
+        const uint32_t sel = (j & 1) ? 0x7632 : 0x5410;   // column j of two keys
+        window_mma(acc[i][j], pa0, pa2, __byte_perm(v0[j >> 1], v1[j >> 1], sel),
+                   __byte_perm(v2[j >> 1], v3[j >> 1], sel));
+      }
+    }
+  };
+  for (int i0 = k_begin + warp * 16; i0 < k_end; i0 += GROUPS * 16) {
+    auto at = [&](int x) -> long long {
+      const int i = i0 + x;
+      return i >= k_end ? -1 : i < n_keep ? i : lo + (i - n_keep);
+    };
+    auto in = [&](const T* base, int pitch, int x) -> const T* {
+      const long long j = at(x);
+      return j < 0 ? nullptr : base + j * pitch;
+    };
+    absorb([&](int x) { return in(kc, p.dimp, x); }, [&](int x) { return in(vc, p.vdimp, x); });
+  }
+  if constexpr (FUSED) {
+    if (rank == 0 && warp == 0)
+      absorb([&](int x) -> const T* { return x ? nullptr : k_new; },
+             [&](int x) -> const T* { return x ? nullptr : v_new; });
+  }
+  l += __shfl_xor_sync(0xffffffffu, l, 1);
+  l += __shfl_xor_sync(0xffffffffu, l, 2);
+  if (c == 0) {
+    mrg[(warp * R + gr) * 2] = m;
+    mrg[(warp * R + gr) * 2 + 1] = l;
+  }
+#pragma unroll
+  for (int i = 0; i < VI; ++i)
+#pragma unroll
+    for (int j = 0; j < 8; ++j)
+#pragma unroll
+      for (int e = 0; e < 2; ++e) {
+        const int col = (2 * c + e + 8 * i) * 8 + j;
+        if (col < DP) acc_s[(warp * R + gr) * DP + col] = acc[i][j][e];
+      }
+  window_finish<T, GROUPS, R, DP>(p, cluster, mrg, acc_s, fin, row, h0, nr, rank);
+}
+
+static int win_start(void (*kern)(const AttnWindowParams), const AttnWindowParams& p, int heads,
+                     size_t smem, cudaStream_t stream) {
+  const int per_g = p.H / p.G, n_rb = (per_g + heads - 1) / heads;
   cudaLaunchConfig_t cfg;
   memset(&cfg, 0, sizeof(cfg));
   cfg.gridDim = dim3(p.splits, p.G * n_rb, p.n);
@@ -487,18 +722,36 @@ static int win_launch(const AttnWindowParams& p, cudaStream_t stream) {
   }
   cfg.attrs = attrs;
   cfg.numAttrs = na;
-  return (int)cudaLaunchKernelEx(&cfg, attn_window_kernel<T, LPK, R, FUSED>, p);
+  return (int)cudaLaunchKernelEx(&cfg, kern, p);
 }
 
-template <typename T, int LPK>
-static int win_pick(const AttnWindowParams& p, bool fused, cudaStream_t stream) {
+template <int LPK, int R, bool FUSED>
+static int win_launch(const AttnWindowParams& p, cudaStream_t stream) {
+  constexpr int GROUPS = kWinThreads / LPK;
+  constexpr size_t smem = sizeof(float) * (R * LPK * 8 + 2 * LPK * 8 + GROUPS * R * 2 +
+                                           GROUPS * R * LPK * 8);
+  static_assert(smem < 48 * 1024, "fits the default limit");
+  return win_start(attn_window_kernel<float, LPK, R, FUSED>, p, R, smem, stream);
+}
+
+template <int LPK, bool FUSED>
+static int win_launch_mma(const AttnWindowParams& p, cudaStream_t stream) {
+  constexpr int R = 8, DP = LPK * 8, GROUPS = kWinThreads / 32;
+  constexpr size_t smem = sizeof(float) * (GROUPS * R * 2 + GROUPS * R * DP) + 2 * (R + 2) * DP;
+  static_assert(smem < 48 * 1024, "fits the default limit");
+  return win_start(attn_window_mma_kernel<LPK, FUSED>, p, R, smem, stream);
+}
+
+template <int LPK>
+static int win_pick(const AttnWindowParams& p, bool fused, bool bf16, cudaStream_t stream) {
   const int per_g = p.H / p.G;
-#define E2H_WIN(R_) return fused ? win_launch<T, LPK, R_, true>(p, stream) \
-                                 : win_launch<T, LPK, R_, false>(p, stream)
+  if (bf16)
+    return fused ? win_launch_mma<LPK, true>(p, stream) : win_launch_mma<LPK, false>(p, stream);
+#define E2H_WIN(R_) return fused ? win_launch<LPK, R_, true>(p, stream) \
+                                 : win_launch<LPK, R_, false>(p, stream)
   if (per_g == 1) E2H_WIN(1);
   if (per_g == 2) E2H_WIN(2);
-  if (per_g <= 4) E2H_WIN(4);
-  E2H_WIN(8);
+  E2H_WIN(4);
 #undef E2H_WIN
 }
 
@@ -561,14 +814,11 @@ extern "C" int e2h_attn_window(const e2h::AttnWindowParams* p, int fused, int is
     q.pos = p->pos + t0;
     q.slot = p->slot + t0;
     q.act = static_cast<char*>(p->act) + (long long)t0 * p->ld * (is_bf16 ? 2 : 4);
-#define E2H_WIN_T(T_)                                          \
-    r = big <= 32 ? win_pick<T_, 4>(q, fused != 0, stream)     \
-        : big <= 64 ? win_pick<T_, 8>(q, fused != 0, stream)   \
-        : big <= 128 ? win_pick<T_, 16>(q, fused != 0, stream) \
-                     : win_pick<T_, 32>(q, fused != 0, stream)
-    if (is_bf16) E2H_WIN_T(__nv_bfloat16);
-    else E2H_WIN_T(float);
-#undef E2H_WIN_T
+    const bool bf = is_bf16 != 0;
+    r = big <= 32    ? win_pick<4>(q, fused != 0, bf, stream)
+        : big <= 64  ? win_pick<8>(q, fused != 0, bf, stream)
+        : big <= 128 ? win_pick<16>(q, fused != 0, bf, stream)
+                     : win_pick<32>(q, fused != 0, bf, stream);
     if (r) return r;
   }
   return 0;

@@ -18,7 +18,7 @@
 //                   tensor-memory operand of S^T q without passing through shared memory:
 //                       S^T += V^T K        (128 x dim,  k = 64 tokens, 2 parts)
 //                       O^T  = V^T A^T + S^T Q^T   (128 x 64 tokens, 2 + 3 part products)
-//                   Roles: TMA producer, tcgen05 issuer, four state warps, four output warps.
+//                   Roles: TMA producer, tcgen05 issuer, eight state warps, four output warps.
 //
 // All mbarrier waits are bounded; a time-out sets the status word, the CTA stops issuing copies,
 // waits (bounded) for those in flight, reaches its barriers and frees its tensor memory.
@@ -302,7 +302,7 @@ __global__ void __launch_bounds__(kPrepThreads, 2) gla_chunk_prep_kernel(const E
 }
 
 // ---------------------------------------------------------------------------------------------
-constexpr int kGsThreads = 320;
+constexpr int kGsThreads = 448;      // producer, issuer, eight state warps, four output warps
 constexpr int kGsStages = 2;
 
 struct GlaCtrl {
@@ -349,7 +349,7 @@ gla_chunk_scan_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
       mbar_init(smem_u32(&ctrl->full[s]), 1);
       mbar_init(smem_u32(&ctrl->empty[s]), 1);
     }
-    mbar_init(smem_u32(&ctrl->s_ready), 4);
+    mbar_init(smem_u32(&ctrl->s_ready), 8);
     mbar_init(smem_u32(&ctrl->s_full), 1);
     for (int s = 0; s < 2; ++s) {
       mbar_init(smem_u32(&ctrl->o_full[s]), 1);
@@ -459,14 +459,15 @@ gla_chunk_scan_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
       umma_commit(smem_u32(&ctrl->empty[s]));
       umma_commit(smem_u32(&ctrl->o_full[b]));
     }
-  } else if (warp >= 2 && warp < 6) {
-    // ---------------- state warps: lane = value column ----------------
+  } else if (warp >= 2 && warp < 10) {
+    // ---------------- state warps: lane = value column, two warps share the key channels --------
     const int q = warp & 3;
+    const int d_lo = (warp - 2) >> 2 ? DP / 2 : 0, d_hi = d_lo + DP / 2;
     const int row = q * 32 + lane;
     const uint32_t lane_off = static_cast<uint32_t>(q * 32) << 16;
     const int col = v0 + row;
     const bool live = col < p.vp;
-    const int st_tid = threadIdx.x - 64;               // 0..127
+    const int st_tid = threadIdx.x - 64;               // 0..255
     float* S = p.state + ((long long)slot * p.H + head) * p.dim * p.vp + col;
     const bool fresh = p.pos[t_begin] == 0;
     auto g_fetch = [&](int c) {
@@ -483,11 +484,11 @@ gla_chunk_scan_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
         ok = __all_sync(0xffffffffu, ok);
         tc_fence_after();
       }
-      asm volatile("bar.sync 1, 128;" ::: "memory");   // g_s of this chunk is written
+      asm volatile("bar.sync 1, 256;" ::: "memory");   // g_s of this chunk is written
       if (c + 1 < n_ch) g_fetch(c + 1);
       const float* g = g_s + (c & 1) * DP;
 #pragma unroll 1
-      for (int d0 = 0; d0 < DP; d0 += 32) {
+      for (int d0 = d_lo; d0 < d_hi; d0 += 32) {
         float v[32];
         if (c == 0) {
 #pragma unroll
@@ -529,7 +530,7 @@ gla_chunk_scan_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
       __syncwarp();
       if (lane == 0) mbar_arrive(smem_u32(&ctrl->s_ready));
     }
-  } else if (warp >= 6) {
+  } else if (warp >= 10) {
     // ---------------- output warps: lane = value column, register = token ----------------
     const int q = warp & 3;
     const int col = v0 + q * 32 + lane;

@@ -62,7 +62,7 @@ def window_splits(n: int, heads: int, kv_heads: int, keys: int) -> int:
     per_g = heads // kv_heads
     ctas = n * kv_heads * -(-per_g // 8)
     s = 1
-    while s < 8 and ctas * s * 2 <= N_SM * 8 and keys // (s * 2) >= 64:
+    while s < 8 and ctas * s * 2 <= N_SM * 4 and keys // (s * 2) >= 64:
         s *= 2
     return s
 
