@@ -251,8 +251,9 @@ __global__ void __launch_bounds__(kScanThreads) gla_scan_kernel(const E2hGlaPara
   }
 }
 
-// One warp per (token, head).
-template <typename T>
+// One warp per (token, head). NV > 0: value columns in multiples of 4, at most NV x 128, whose
+// output and gate are fetched at once; 0: any size.
+template <typename T, int NV>
 __global__ void __launch_bounds__(256) gla_out_kernel(const E2hGlaParams p) {
   pdl_launch_dependents();
   pdl_wait_prior();
@@ -264,34 +265,51 @@ __global__ void __launch_bounds__(256) gla_out_kernel(const E2hGlaParams p) {
   const float* o = p.o + w * p.vdim;
   T* g = static_cast<T*>(p.act) + t * p.ld + p.off_g + (long long)head * p.vdim;
   float ss = 0.f;
-  if ((p.vdim & 3) == 0 && (p.ld & 3) == 0 && (p.off_g & 3) == 0) {   // 4 columns per access
-    for (int i = lane * 4; i < p.vdim; i += 128) {
-      float x[4];
-      load4(o + i, x);
-      ss += x[0] * x[0] + x[1] * x[1] + x[2] * x[2] + x[3] * x[3];
-    }
+  if constexpr (NV > 0) {
+    float x[NV][4], z[NV][4];
 #pragma unroll
-    for (int m = 16; m > 0; m >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, m);
+    for (int k = 0; k < NV; ++k) {
+      const int i = lane * 4 + k * 128;
+      if (i < p.vdim) {
+        load4(o + i, x[k]);
+        load4(g + i, z[k]);
+#pragma unroll
+        for (int e = 0; e < 4; ++e) ss += x[k][e] * x[k][e];
+      }
+    }
+    ss = warp_sum(ss);
     const float rstd = 1.f / sqrtf(ss / p.vdim + p.eps);
-    for (int i = lane * 4; i < p.vdim; i += 128) {
-      float x[4], z[4], w[4];
-      load4(o + i, x);
-      load4(g + i, z);
-      load4(p.norm + i, w);
 #pragma unroll
-      for (int e = 0; e < 4; ++e) x[e] = x[e] * rstd * w[e] * (z[e] * sigmoid_f(z[e]));
-      store4(g + i, x);
+    for (int k = 0; k < NV; ++k) {
+      const int i = lane * 4 + k * 128;
+      if (i < p.vdim) {
+        float wt[4];
+        load4(p.norm + i, wt);
+#pragma unroll
+        for (int e = 0; e < 4; ++e) x[k][e] *= rstd * wt[e] * (z[k][e] * sigmoid_f(z[k][e]));
+        store4(g + i, x[k]);
+      }
     }
-    return;
+  } else {
+    for (int i = lane; i < p.vdim; i += 32) ss += o[i] * o[i];
+    ss = warp_sum(ss);
+    const float rstd = 1.f / sqrtf(ss / p.vdim + p.eps);
+    for (int i = lane; i < p.vdim; i += 32) {
+      const float z = to_f(g[i]);
+      g[i] = from_f<T>(o[i] * rstd * p.norm[i] * (z * sigmoid_f(z)));
+    }
   }
-  for (int i = lane; i < p.vdim; i += 32) ss += o[i] * o[i];
-#pragma unroll
-  for (int m = 16; m > 0; m >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, m);
-  const float rstd = 1.f / sqrtf(ss / p.vdim + p.eps);
-  for (int i = lane; i < p.vdim; i += 32) {
-    const float z = to_f(g[i]);
-    g[i] = from_f<T>(o[i] * rstd * p.norm[i] * (z * sigmoid_f(z)));
-  }
+}
+
+template <typename T>
+static int gla_out(const E2hGlaParams& p, cudaStream_t s) {
+  const long long warps = (long long)p.n * p.H;
+  const dim3 grid((unsigned)((warps + 7) / 8));
+  const bool vec = (p.vdim & 3) == 0 && (p.ld & 3) == 0 && (p.off_g & 3) == 0;
+  if (vec && p.vdim <= 128) return (int)launch(gla_out_kernel<T, 1>, grid, dim3(256), 0, s, p);
+  if (vec && p.vdim <= 256) return (int)launch(gla_out_kernel<T, 2>, grid, dim3(256), 0, s, p);
+  if (vec && p.vdim <= 512) return (int)launch(gla_out_kernel<T, 4>, grid, dim3(256), 0, s, p);
+  return (int)launch(gla_out_kernel<T, 0>, grid, dim3(256), 0, s, p);
 }
 
 static int gla_check(const E2hGlaParams& p) {
@@ -380,12 +398,8 @@ int e2h_gla_out(const E2hGlaParams* p, int is_bf16, void* stream) {
   int r = gla_check(*p);
   if (r) return r;
   if (!p->o) return -1;
-  const long long warps = (long long)p->n * p->H;
-  const dim3 grid((unsigned)((warps + 7) / 8));
-  return is_bf16 ? (int)launch(gla_out_kernel<__nv_bfloat16>, grid, dim3(256), 0,
-                               (cudaStream_t)stream, *p)
-                 : (int)launch(gla_out_kernel<float>, grid, dim3(256), 0, (cudaStream_t)stream,
-                               *p);
+  return is_bf16 ? gla_out<__nv_bfloat16>(*p, (cudaStream_t)stream)
+                 : gla_out<float>(*p, (cudaStream_t)stream);
 }
 
 }  // extern "C"

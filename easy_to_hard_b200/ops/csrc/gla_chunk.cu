@@ -43,20 +43,33 @@ constexpr float kSteep = 40.f;         // decay (in e) up to which its inverse i
 __device__ __forceinline__ int chunk_place(const E2hGlaParams& p, int sg, int c) {
   return p.seg[sg] / kC + sg + c;
 }
+__device__ __forceinline__ float exp_ftz(float x) { return ex2_approx(x * 1.4426950408889634f); }
+__device__ __forceinline__ float lg2_ftz(float x) {
+  float y;
+  asm("lg2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+__device__ __forceinline__ float rcp_ftz(float x) {
+  float y;
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
 // log sigmoid(z) to about 1e-7 absolute: it is only ever added up and exponentiated
 __device__ __forceinline__ float log_sigmoid_c(float z) {
-  const float e = __expf(-fabsf(z));
+  const float e = exp_ftz(-fabsf(z));
   // log(1 + e): Taylor series where 1 + e would round e away
-  const float l = e < 0.03f ? e * (1.f - e * (0.5f - e * (1.f / 3.f - e * 0.25f))) : __logf(1.f + e);
+  const float l = e < 0.03f ? e * (1.f - e * (0.5f - e * (1.f / 3.f - e * 0.25f)))
+                            : lg2_ftz(1.f + e) * 0.6931471805599453f;
   return fminf(z, 0.f) - l;
-}
-__device__ __forceinline__ void split_bf16(float x, float& hi, float& lo) {
-  hi = bf16_round(x);
-  lo = x - hi;
 }
 __device__ __forceinline__ uint32_t pack2(float a, float b) {
   const __nv_bfloat162 v = __floats2bfloat162_rn(a, b);
   return *reinterpret_cast<const uint32_t*>(&v);
+}
+// two values as packed bf16 high parts and packed bf16 low parts
+__device__ __forceinline__ void split2(float a, float b, uint32_t& hi, uint32_t& lo) {
+  hi = pack2(a, b);
+  lo = pack2(a - __uint_as_float(hi << 16), b - __uint_as_float(hi & 0xffff0000u));
 }
 __device__ __forceinline__ void mma_16816(float* c, const uint32_t* a, const uint32_t* b) {
   asm volatile(
@@ -66,19 +79,43 @@ __device__ __forceinline__ void mma_16816(float* c, const uint32_t* a, const uin
       : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b[0]), "r"(b[1]));
 }
 
-constexpr int kPrepThreads = 256;
+constexpr int kPrepThreads = 512;
 constexpr int kAT = kC + 4;            // row pitch of the transposed decay input
 
 __host__ __device__ inline int prep_smem_bytes(int dim, int r) {
   // b [64][dim + 4] fp32, four bf16 [64][dim + 8] (q and k in two parts), a^T [r][68] fp32,
-  // partial sums [256]
-  return kC * (dim + 4) * 4 + 4 * kC * (dim + 8) * 2 + r * kAT * 4 + kPrepThreads * 4;
+  // partial sums [512], decay of the whole chunk [dim]
+  return kC * (dim + 4) * 4 + 4 * kC * (dim + 8) * 2 + r * kAT * 4 + kPrepThreads * 4 + dim * 4;
 }
 
-// 16 x 16 blocks (row, column) of A by warp; those above the diagonal are zero
-__constant__ unsigned char kPrepBlocks[8][2] = {{0x30, 0x31}, {0x32, 0x33}, {0x20, 0x21},
-                                                {0x22, 0x01}, {0x10, 0x11}, {0x00, 0x02},
-                                                {0x03, 0x12}, {0x13, 0x23}};
+// Decay logits of J x 4 consecutive tokens (from tb on) of one key channel: w . a_t + bias.
+template <int J>
+__device__ __forceinline__ void decay_logits(float* z, const __nv_bfloat16* w, bool wvec, int r,
+                                             const float* at, float bias) {
+#pragma unroll
+  for (int j = 0; j < 4 * J; ++j) z[j] = bias;
+  for (int i0 = 0; i0 < r; i0 += 8) {
+    float wv[8];
+    if (wvec) {
+      load8(w + i0, wv);
+    } else {
+#pragma unroll
+      for (int e = 0; e < 8; ++e) wv[e] = i0 + e < r ? to_f(w[i0 + e]) : 0.f;
+    }
+#pragma unroll
+    for (int e = 0; e < 8; ++e) {
+      if (i0 + e >= r) break;
+#pragma unroll
+      for (int j = 0; j < J; ++j) {
+        const float4 av = *reinterpret_cast<const float4*>(at + (i0 + e) * kAT + 4 * j);
+        z[4 * j] = fmaf(wv[e], av.x, z[4 * j]);
+        z[4 * j + 1] = fmaf(wv[e], av.y, z[4 * j + 1]);
+        z[4 * j + 2] = fmaf(wv[e], av.z, z[4 * j + 2]);
+        z[4 * j + 3] = fmaf(wv[e], av.w, z[4 * j + 3]);
+      }
+    }
+  }
+}
 
 // MMA fragments of rows r0.. and columns k0.. of a [64][pitch] bf16 tile
 __device__ __forceinline__ uint32_t frag(const __nv_bfloat16* x, int row, int col, int pitch) {
@@ -94,7 +131,8 @@ __global__ void __launch_bounds__(kPrepThreads, 2) gla_chunk_prep_kernel(const E
   __nv_bfloat16* kh_s = ql_s + kC * LQ;
   __nv_bfloat16* kl_s = kh_s + kC * LQ;
   float* at_s = reinterpret_cast<float*>(kl_s + kC * LQ);                 // [r][kAT]
-  float* sum_s = at_s + p.r * kAT;                                        // [256]
+  float* sum_s = at_s + p.r * kAT;                                        // [512]
+  float* g_s = sum_s + kPrepThreads;                                      // [dim]
   pdl_launch_dependents();
   pdl_wait_prior();
   const int c = blockIdx.x, head = blockIdx.y, sg = blockIdx.z;
@@ -108,6 +146,19 @@ __global__ void __launch_bounds__(kPrepThreads, 2) gla_chunk_prep_kernel(const E
     return;
   }
   const int tid = threadIdx.x;
+  const __nv_bfloat16* act = static_cast<const __nv_bfloat16*>(p.act) + (long long)t0 * p.ld +
+                             (long long)head * D;
+  // the thread's q and k (at most 2 pieces of 8 columns): in flight under the decays
+  uint4 q4[2], k4[2];
+#pragma unroll
+  for (int n = 0; n < 2; ++n) {
+    const int i = tid + n * kPrepThreads, t = i / (D / 8), d = (i - t * (D / 8)) * 8;
+    q4[n] = k4[n] = make_uint4(0, 0, 0, 0);
+    if (t < nt) {
+      q4[n] = *reinterpret_cast<const uint4*>(act + (long long)t * p.ld + p.off_q + d);
+      k4[n] = *reinterpret_cast<const uint4*>(act + (long long)t * p.ld + p.off_k + d);
+    }
+  }
   for (int i = tid; i < kC * p.r; i += kPrepThreads) {
     const int t = i / p.r, k = i - t * p.r;
     at_s[k * kAT + t] = t < nt ? p.a[(long long)(t0 + t) * p.lda + k] : 0.f;
@@ -115,10 +166,10 @@ __global__ void __launch_bounds__(kPrepThreads, 2) gla_chunk_prep_kernel(const E
   __syncthreads();
   // running sums of log alpha: `ng` groups of threads take consecutive runs of tokens of a column
   {
-    const int ng = min(kPrepThreads / D, 16), run = ((kC + ng - 1) / ng + 3) / 4 * 4;   // <= 32
+    const int ng = min(kPrepThreads / D, 16), run = ((kC + ng - 1) / ng + 3) / 4 * 4;   // <= 16
     const int g = tid / D, d = tid - g * D, tb = g * run;
     const bool work = g < ng && tb < kC;
-    float z[32];
+    float z[16];
     float add = 0.f;
     if (work) {
       const __nv_bfloat16* w = static_cast<const __nv_bfloat16*>(p.w2) +
@@ -126,34 +177,13 @@ __global__ void __launch_bounds__(kPrepThreads, 2) gla_chunk_prep_kernel(const E
       const bool wvec = (p.ldw & 7) == 0 && (p.r & 7) == 0 &&
                         (reinterpret_cast<uintptr_t>(p.w2) & 15) == 0;
       const float bias = p.b2[head * D + d];
-#pragma unroll
-      for (int j = 0; j < 32; ++j) z[j] = bias;
-      for (int i0 = 0; i0 < p.r; i0 += 8) {
-        float wv[8];
-        if (wvec) {
-          load8(w + i0, wv);
-        } else {
-#pragma unroll
-          for (int e = 0; e < 8; ++e) wv[e] = i0 + e < p.r ? to_f(w[i0 + e]) : 0.f;
-        }
-#pragma unroll
-        for (int e = 0; e < 8; ++e) {
-          if (i0 + e >= p.r) break;
-          const float* at = at_s + (i0 + e) * kAT + tb;
-#pragma unroll
-          for (int j = 0; j < 8; ++j) {
-            if (4 * j >= run) break;
-            const float4 av = *reinterpret_cast<const float4*>(at + 4 * j);
-            z[4 * j] = fmaf(wv[e], av.x, z[4 * j]);
-            z[4 * j + 1] = fmaf(wv[e], av.y, z[4 * j + 1]);
-            z[4 * j + 2] = fmaf(wv[e], av.z, z[4 * j + 2]);
-            z[4 * j + 3] = fmaf(wv[e], av.w, z[4 * j + 3]);
-          }
-        }
-      }
+      // a run of 12 computes 16: the columns read past the row are in shared memory, not used
+      if (run == 4) decay_logits<1>(z, w, wvec, p.r, at_s + tb, bias);
+      else if (run == 8) decay_logits<2>(z, w, wvec, p.r, at_s + tb, bias);
+      else decay_logits<4>(z, w, wvec, p.r, at_s + tb, bias);
       float acc = 0.f;
 #pragma unroll
-      for (int j = 0; j < 32; ++j) {
+      for (int j = 0; j < 16; ++j) {
         if (j < run && tb + j < nt) acc += log_sigmoid_c(z[j]) * p.inv_tau;
         z[j] = acc;
       }
@@ -163,7 +193,7 @@ __global__ void __launch_bounds__(kPrepThreads, 2) gla_chunk_prep_kernel(const E
     if (work) {
       for (int k = 0; k < g; ++k) add += sum_s[k * D + d];
 #pragma unroll
-      for (int j = 0; j < 32; ++j)
+      for (int j = 0; j < 16; ++j)
         if (j < run && tb + j < kC) b_s[(tb + j) * LB + d] = z[j] + add;
     }
   }
@@ -172,51 +202,38 @@ __global__ void __launch_bounds__(kPrepThreads, 2) gla_chunk_prep_kernel(const E
   bool mine = false;
   for (int d = tid; d < D; d += kPrepThreads) {
     mine = mine || !(-b_end[d] <= kSteep);
-    p.cg[((long long)place * p.H + head) * D + d] = __expf(b_end[d]);
+    g_s[d] = exp_ftz(b_end[d]);
+    p.cg[((long long)place * p.H + head) * D + d] = g_s[d];
   }
   // steep: the inverse decay of the chunk leaves the fp32 range; A then takes its exact form and
   // the shared tiles hold the plain q and k
   const bool steep = __syncthreads_or(mine) != 0;
-  const __nv_bfloat16* act = static_cast<const __nv_bfloat16*>(p.act) + (long long)t0 * p.ld +
-                             (long long)head * D;
   const long long row0 = ((long long)place * p.H + head) * kC;
   const long long part = (long long)p.chunks * p.H * kC * D;
   __nv_bfloat16* cq = static_cast<__nv_bfloat16*>(p.cq) + row0 * D;
   __nv_bfloat16* ck = static_cast<__nv_bfloat16*>(p.ck) + row0 * D;
-  for (int i = tid; i < kC * (D / 8); i += kPrepThreads) {
-    const int t = i / (D / 8), d = (i - t * (D / 8)) * 8;
-    float q[8], k[8], b[8];
-    if (t < nt) {
-      load8(act + (long long)t * p.ld + p.off_q + d, q);
-      load8(act + (long long)t * p.ld + p.off_k + d, k);
-    } else {
 #pragma unroll
-      for (int e = 0; e < 8; ++e) q[e] = k[e] = 0.f;
-    }
+  for (int n = 0; n < 2; ++n) {
+    const int i = tid + n * kPrepThreads, t = i / (D / 8), d = (i - t * (D / 8)) * 8;
+    if (t >= kC) break;
+    float q[8], k[8], b[8];
+    load8(reinterpret_cast<const __nv_bfloat16*>(&q4[n]), q);
+    load8(reinterpret_cast<const __nv_bfloat16*>(&k4[n]), k);
     load8(b_s + t * LB + d, b);
     uint32_t qh[4], ql[4], kh[4], kl[4], eh[4], el[4];
+    float gd[8];
+    load8(g_s + d, gd);
 #pragma unroll
     for (int e = 0; e < 8; e += 2) {
-      float h[2], l[2], ih[2], il[2], xh[2], xl[2];
-#pragma unroll
-      for (int u = 0; u < 2; ++u) {
-        const float eb = __expf(b[e + u]);
-        split_bf16(q[e + u] * p.qscale * eb, h[u], l[u]);
-        if (!steep) {
-          const float ki = __fdividef(k[e + u], eb);
-          split_bf16(ki, ih[u], il[u]);
-          split_bf16(ki * __expf(b_end[d + e + u]), xh[u], xl[u]);
-        } else {
-          split_bf16(k[e + u] * __expf(b_end[d + e + u] - b[e + u]), xh[u], xl[u]);
-        }
-      }
-      qh[e / 2] = pack2(h[0], h[1]);
-      ql[e / 2] = pack2(l[0], l[1]);
-      eh[e / 2] = pack2(xh[0], xh[1]);
-      el[e / 2] = pack2(xl[0], xl[1]);
+      const float e0 = exp_ftz(b[e]), e1 = exp_ftz(b[e + 1]);
+      split2(q[e] * p.qscale * e0, q[e + 1] * p.qscale * e1, qh[e / 2], ql[e / 2]);
       if (!steep) {
-        kh[e / 2] = pack2(ih[0], ih[1]);
-        kl[e / 2] = pack2(il[0], il[1]);
+        const float k0 = k[e] * rcp_ftz(e0), k1 = k[e + 1] * rcp_ftz(e1);
+        split2(k0, k1, kh[e / 2], kl[e / 2]);
+        split2(k0 * gd[e], k1 * gd[e + 1], eh[e / 2], el[e / 2]);
+      } else {
+        split2(k[e] * exp_ftz(b_end[d + e] - b[e]), k[e + 1] * exp_ftz(b_end[d + e + 1] - b[e + 1]),
+               eh[e / 2], el[e / 2]);
       }
     }
     const long long o = (long long)t * D + d;
@@ -244,8 +261,8 @@ __global__ void __launch_bounds__(kPrepThreads, 2) gla_chunk_prep_kernel(const E
   const int gr = lane >> 2, c2 = (lane & 3) * 2;
   __nv_bfloat16* ca = static_cast<__nv_bfloat16*>(p.ca) + row0 * kC;
   const long long apart = (long long)p.chunks * p.H * kC * kC;
-  for (int n = 0; n < 2; ++n) {
-    const int bi = kPrepBlocks[warp][n] >> 4, bj = kPrepBlocks[warp][n] & 15;
+  {
+    const int bi = warp >> 2, bj = warp & 3;      // one block per warp, those above the diagonal 0
     float acc[2][4];
 #pragma unroll
     for (int x = 0; x < 2; ++x)
@@ -283,7 +300,7 @@ __global__ void __launch_bounds__(kPrepThreads, 2) gla_chunk_prep_kernel(const E
           float v = 0.f;
           for (int d = 0; d < D; ++d)
             v = fmaf(to_f(qh_s[t * LQ + d]) * p.qscale,
-                     to_f(kh_s[s * LQ + d]) * __expf(b_s[t * LB + d] - b_s[s * LB + d]), v);
+                     to_f(kh_s[s * LQ + d]) * exp_ftz(b_s[t * LB + d] - b_s[s * LB + d]), v);
           acc[nb][y] = v;
         }
     }
@@ -292,11 +309,10 @@ __global__ void __launch_bounds__(kPrepThreads, 2) gla_chunk_prep_kernel(const E
 #pragma unroll
       for (int hf = 0; hf < 2; ++hf) {
         const int t = 16 * bi + gr + hf * 8, s = 16 * bj + nb * 8 + c2;
-        float h0, l0, h1, l1;
-        split_bf16(s <= t ? acc[nb][2 * hf] : 0.f, h0, l0);
-        split_bf16(s + 1 <= t ? acc[nb][2 * hf + 1] : 0.f, h1, l1);
-        *reinterpret_cast<uint32_t*>(ca + t * kC + s) = pack2(h0, h1);
-        *reinterpret_cast<uint32_t*>(ca + apart + t * kC + s) = pack2(l0, l1);
+        uint32_t hi, lo;
+        split2(s <= t ? acc[nb][2 * hf] : 0.f, s + 1 <= t ? acc[nb][2 * hf + 1] : 0.f, hi, lo);
+        *reinterpret_cast<uint32_t*>(ca + t * kC + s) = hi;
+        *reinterpret_cast<uint32_t*>(ca + apart + t * kC + s) = lo;
       }
   }
 }
@@ -509,11 +525,7 @@ gla_chunk_scan_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
         uint32_t hi[16], lo[16];
 #pragma unroll
         for (int i = 0; i < 16; ++i) {
-          float h0, l0, h1, l1;
-          split_bf16(v[2 * i], h0, l0);
-          split_bf16(v[2 * i + 1], h1, l1);
-          hi[i] = pack2(h0, h1);
-          lo[i] = pack2(l0, l1);
+          split2(v[2 * i], v[2 * i + 1], hi[i], lo[i]);
           v[2 * i] *= g[d0 + 2 * i];
           v[2 * i + 1] *= g[d0 + 2 * i + 1];
         }
