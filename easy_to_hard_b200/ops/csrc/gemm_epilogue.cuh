@@ -93,6 +93,24 @@ __device__ __forceinline__ void epilogue8(const E2hGemmParams& p, int f, int t0,
           asm volatile("red.relaxed.gpu.global.add.f32 [%0], %1;" ::"l"(
                            out + (long long)(t0 + j) * p.ldo + f), "f"(v[j]) : "memory");
     } break;
+    case E2H_EPI_RESIDUAL: {
+      __nv_bfloat16* out = static_cast<__nv_bfloat16*>(p.out);
+      const __nv_bfloat16* res = static_cast<const __nv_bfloat16*>(p.aux);
+      // all residual loads first: `out` may alias `res`, so a load placed after a store could
+      // not be moved above it and the eight round trips would run one after another
+      float r[8];
+#pragma unroll
+      for (int j = 0; j < 8; ++j) {
+        const int t = t0 + j;
+        r[j] = (f_ok && t < t_end) ? __bfloat162float(res[(long long)t * p.ldo + f]) : 0.f;
+      }
+#pragma unroll
+      for (int j = 0; j < 8; ++j) {
+        const int t = t0 + j;
+        if (f_ok && t < t_end)
+          out[(long long)t * p.ldo + f] = __float2bfloat16_rn(bf16_round(v[j]) + r[j]);
+      }
+    } break;
     case E2H_EPI_SWIGLU: {
       if constexpr (DUAL) {
         __nv_bfloat16* out = static_cast<__nv_bfloat16*>(p.out);
