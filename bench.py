@@ -16,6 +16,8 @@ with CUDA events between barriers, max over ranks.
 prompt copied from pinned host memory and the generated tokens copied back to pinned host memory
 inside the timed region of every step.
 
+``--workload bovinex`` measures the hybrid decoder beside the LLaMA path at equal size instead.
+
 ``--impl reference`` runs the unmodified reference from ``baseline/_ref`` (its ``Transformer``,
 ``apply_tp`` and ``generate`` with its ``torch.compile``'d decode step) on the same workload.
 """

@@ -220,6 +220,8 @@ LAYERS = {
     "d64v128": M.attn(8, 1, 64, 128, rot=32, window=64, keep=0),
     "d14": M.attn(3, 1, 14, 10, rot=6, window=9, keep=2),
     "d200": M.attn(2, 1, 200, 256, rot=40, window=100, keep=17),
+    "d56v48": M.attn(6, 2, 56, 48, rot=56, window=150, keep=9),
+    "d96v80": M.attn(4, 4, 96, 80, rot=48, scaling=M.YARN, window=31, keep=140),
     "mqa16": M.attn(16, 1, 72, 96, window=130, keep=129),
 }
 
@@ -389,6 +391,11 @@ GLA = {  # heads, dim, vdim, tau, rank, bias, spread of the decay logits
     "odd": (3, 7, 9, 3.0, 5, 0.0, 1.0),
     "deep": (1, 256, 72, 2.0, 24, 1.0, 2.0),
     "forgets": (2, 64, 64, 1.0, 16, -20.0, 15.0),   # decays from about e^-60 to 1 in one step
+    "half": (2, 48, 48, 8.0, 16, 0.0, 1.0),
+    "tall": (2, 80, 136, 8.0, 5, 0.0, 1.0),         # decay rank off the vector width
+    "flat": (1, 112, 40, 16.0, 20, 1.0, 1.0),
+    "thin": (4, 16, 264, 4.0, 16, 0.0, 1.0),
+    "edge": (2, 96, 64, 8.0, 16, -5.0, 0.5),        # around the steepest chunk of the fast form
     "keeps": (2, 128, 128, 16.0, 16, 30.0, 0.0),    # nothing decays: the sum over all tokens
 }
 
