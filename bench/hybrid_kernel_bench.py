@@ -71,7 +71,7 @@ def i32(x):
 
 
 def bovinex(size, batch, context, prompts, plen):
-    from easy_to_hard_b200.models.hybrid_engine import _Work
+    from easy_to_hard_b200.models.hybrid_engine import _Scratch
     from easy_to_hard_b200.ops import gemm, hybrid as hy
     model = bovinex_model(size, 4)
     n_max = prompts * plen
@@ -81,7 +81,7 @@ def bovinex(size, batch, context, prompts, plen):
         head(f"Bovinex {size}, {phase}: " + (f"{batch} sequences at position {context}"
                                              if phase == "decode" else
                                              f"{prompts} prompts of {plen} tokens"))
-        w = _Work(model, n)
+        w = _Scratch(model, n)
         w.x.normal_()
         if phase == "decode":
             pos, slot, seg = i32([context] * n), i32(list(range(n))), None

@@ -31,7 +31,7 @@ from .slot_cache import SlotCache
 MAX_FORWARD_TOKENS = 32768
 
 
-class _Work:
+class _Scratch:
     """Activation buffers for up to ``n`` tokens."""
 
     def __init__(self, model: HybridLM, n: int):
@@ -100,12 +100,12 @@ class HybridEngine(GenerationEngine):
         self.tok_pos = torch.zeros(self.B, dtype=torch.int32, device=dev)
         self.logits = torch.zeros(self.B, pad8(self.vocab), dtype=torch.float32, device=dev)
         self.hf = torch.zeros(self.B, pad8(cfg.dim), dtype=model.dtype, device=dev)
-        self._work = _Work(model, self.B)
+        self._scratch = _Scratch(model, self.B)
         self._rows: List[Hashable] = []
         self.layer_trace: Optional[list] = None    # a list collects the residual after each layer
 
     # ------------------------------------------------------------------ forward
-    def _forward(self, w: _Work, n: int, tokens, pos, slot, *, seg=None, rows=None,
+    def _forward(self, w: _Scratch, n: int, tokens, pos, slot, *, seg=None, rows=None,
                  decode_counters: bool = False, hf=None, logits=None) -> None:
         """Runs ``n`` packed tokens through all layers. ``seg`` = (device offsets, segments,
         longest segment), or None when every token is the next one of its own sequence. ``rows``
@@ -161,7 +161,7 @@ class HybridEngine(GenerationEngine):
                 last += (y.float()[place.long()][..., :W] * ew[..., None]).sum(1)
             self.layer_trace.append(last)
 
-    def _experts(self, w: _Work, blk, n: int, hw, tail):
+    def _experts(self, w: _Scratch, blk, n: int, hw, tail):
         f, W = blk.layer.mlp, self.model.config.dim
         place, ew = w.choice(n, f.top)
         k = hy.moe_route(tail[:, blk.off_r:], f.experts, f.top, hw, w.hg[: n * f.top, :W], w.off,
@@ -213,7 +213,7 @@ class HybridEngine(GenerationEngine):
         longest = max(b - a for a, b in zip(seg, seg[1:]))
         packed = torch.tensor(toks + pos + slot + seg + rows, dtype=torch.int32).to(self.dev)
         t_d, p_d, s_d, seg_d, rows_d = packed.split([n, n, n, len(seg), len(rows)])
-        w = self._work if n <= self.B else _Work(self.model, n)
+        w = self._scratch if n <= self.B else _Scratch(self.model, n)
         hf = torch.zeros(len(rows), pad8(self.cfg.dim), dtype=self.model.dtype, device=self.dev)
         logits = torch.empty(len(rows), pad8(self.vocab), dtype=torch.float32, device=self.dev)
         self._forward(w, n, t_d, p_d, s_d, rows=rows_d,
@@ -273,7 +273,7 @@ class HybridEngine(GenerationEngine):
             self.cache.close(self._rows.pop())
 
     def _decode_step(self, B, temperature, top_k, eos_id):
-        self._forward(self._work, B, self.next_tok[:B], self.tok_pos[:B], self.slot[:B],
+        self._forward(self._scratch, B, self.next_tok[:B], self.tok_pos[:B], self.slot[:B],
                       decode_counters=True, hf=self.hf, logits=self.logits)
         self._sample(self.logits[:B], B, temperature, top_k, eos_id)
         self._count(1)
@@ -328,7 +328,7 @@ class HybridEngine(GenerationEngine):
             [n, n, n, len(seg), len(rows), len(fin)])
         tokens = ids.reshape(-1)[cell.long()]
         longest = max(t for _, _, t in pick)
-        w = self._work if n <= self.B else _Work(self.model, n)
+        w = self._scratch if n <= self.B else _Scratch(self.model, n)
         whole = len(fin) == ids.shape[0]
         logits = self.logits if whole else torch.empty_like(self.logits)
         self._forward(w, n, tokens, pos, slot, seg=(seg_d, len(seg) - 1, longest), rows=rows_d,
