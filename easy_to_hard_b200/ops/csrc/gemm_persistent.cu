@@ -31,6 +31,7 @@ constexpr int kPThreads = 192;
 constexpr int kPMaxStages = 8;
 constexpr int kChunkTok = 32;                       // tokens per staged epilogue chunk
 constexpr int kChunkBytes = kChunkTok * 128 * 2;    // [32 tokens][128 features] bf16
+constexpr int kPMaxGroups = 96;                     // matrices of a grouped product
 constexpr int kGroupT = 8;                          // token tiles per scheduling band
 
 struct PCtrl {
@@ -41,7 +42,11 @@ struct PCtrl {
   uint64_t res_full[2];
   uint32_t tmem_base;
   int abort_flag;
+  // grouped products: tiles before group g, first row of group g
+  int g_tiles[kPMaxGroups + 1];
+  int g_row[kPMaxGroups + 1];
 };
+static_assert(sizeof(PCtrl) <= 1024, "the control block has one KiB");
 
 __device__ __forceinline__ void tma_store_2d(const void* tmap, uint32_t src, int x, int y) {
   asm volatile(
@@ -86,6 +91,33 @@ __device__ __forceinline__ void tile_coords(int id, int n_f, int n_t, int& ft, i
   tt = band * kGroupT + r % tb;
 }
 
+// A tile of the walk: feature tile, first token row, end of the token rows it may write, and the row
+// of its weight block in the A operand. A grouped product walks group after group; `g` is the
+// caller's running group (tiles come in ascending order).
+struct PTile {
+  int ft, t0, t_end, a_row;
+};
+template <int BN>
+__device__ __forceinline__ PTile tile_at(const E2hGemmParams& p, const PCtrl* ctrl, int id, int n_f,
+                                         int n_t, int& g) {
+  PTile t;
+  int tt;
+  if (p.n_groups > 0) {
+    while (id >= ctrl->g_tiles[g + 1]) ++g;      // id is below the last entry
+    const int row = ctrl->g_row[g], end = ctrl->g_row[g + 1];
+    tile_coords(id - ctrl->g_tiles[g], n_f, (end - row + BN - 1) / BN, t.ft, tt);
+    t.t0 = row + tt * BN;
+    t.t_end = end;
+    t.a_row = g * p.F;
+  } else {
+    tile_coords(id, n_f, n_t, t.ft, tt);
+    t.t0 = tt * BN;
+    t.t_end = p.T;
+    t.a_row = 0;
+  }
+  return t;
+}
+
 // PAIR: two CTAs of a cluster share one 256 (features) x 256 (tokens) tile with cta_group::2
 // instructions: CTA r of the pair owns features [128 r, 128 r + 128) of the tile (its A rows, its
 // accumulator lanes, its epilogue) and stages the B rows of tokens [128 r, 128 r + 128); the
@@ -122,7 +154,7 @@ umma_gemm_persistent_kernel(const __grid_constant__ CUtensorMap tmA,
   const int n_workers = PAIR ? (int)(gridDim.x >> 1) : (int)gridDim.x;
   constexpr int TILE_F = PAIR ? 256 : 128;
   const int n_f = (p.F + TILE_F - 1) / TILE_F, n_t = (p.T + BN - 1) / BN;
-  const int n_tiles = n_f * n_t;
+  int n_tiles = n_f * n_t;
   const int n_kb = (p.K + 63) / 64;
   volatile int* abort_flag = &ctrl->abort_flag;
 
@@ -159,6 +191,23 @@ umma_gemm_persistent_kernel(const __grid_constant__ CUtensorMap tmA,
   if constexpr (PAIR) cluster_sync_all();   // the peer's barriers exist before anything signals them
   pdl_wait_prior();
   pdl_launch_dependents();
+  if (p.n_groups > 0) {                     // the offsets come from the predecessor
+    if (threadIdx.x == 0) {
+      int tiles_ = 0, row = 0;
+      for (int g = 0; g < p.n_groups; ++g) {
+        int end = p.group_off[g + 1];
+        end = end < row ? row : end > p.T ? p.T : end;
+        ctrl->g_tiles[g] = tiles_;
+        ctrl->g_row[g] = row;
+        tiles_ += n_f * ((end - row + BN - 1) / BN);
+        row = end;
+      }
+      ctrl->g_tiles[p.n_groups] = tiles_;
+      ctrl->g_row[p.n_groups] = row;
+    }
+    __syncthreads();
+    n_tiles = ctrl->g_tiles[p.n_groups];
+  }
 
   if (warp == 0 && lane == 0) {
     // ---------------- TMA producer ----------------
@@ -169,11 +218,12 @@ umma_gemm_persistent_kernel(const __grid_constant__ CUtensorMap tmA,
     const uint32_t full0 = smem_u32(&ctrl->full[0]), empty0 = smem_u32(&ctrl->empty[0]);
     const uint32_t tiles0 = smem_u32(tiles);
     bool ok = true;
+    int grp = 0;
     const uint32_t full_lead0 = PAIR ? mapa_shared(full0, 0) : full0;   // leader's full barriers
     for (int tile = worker; tile < n_tiles && ok; tile += n_workers) {
-      int ft, tt;
-      tile_coords(tile, n_f, n_t, ft, tt);
-      const int f0 = ft * TILE_F + crank * 128, t0 = tt * BN + crank * BROWS * (PAIR ? 1 : 0);
+      const PTile pt = tile_at<BN>(p, ctrl, tile, n_f, n_t, grp);
+      const int f0 = pt.a_row + pt.ft * TILE_F + crank * 128;
+      const int t0 = pt.t0 + crank * BROWS * (PAIR ? 1 : 0);
       for (int kb = 0; kb < n_kb; ++kb, ++it) {
         if (!mbar_wait(empty0 + 8 * s, ph ^ 1, abort_flag, p.status, kStatusTimeoutEmpty)) {
           ok = false;
@@ -303,15 +353,14 @@ umma_gemm_persistent_kernel(const __grid_constant__ CUtensorMap tmA,
     const int et = threadIdx.x - 64;                    // 0..127 among the epilogue threads
     const uint32_t taddr = tmem_base + (static_cast<uint32_t>(q * 32) << 16);
     const bool with_res = staged && p.epi == E2H_EPI_RESIDUAL;
-    int tcount = 0, cc = 0;
+    int tcount = 0, cc = 0, grp = 0;
     bool ok = true;
     // the accumulator goes back to the MMA thread of the pair's leader
     const uint32_t tmem_empty0 = PAIR ? mapa_shared(smem_u32(&ctrl->tmem_empty[0]), 0)
                                       : smem_u32(&ctrl->tmem_empty[0]);
     for (int tile = worker; tile < n_tiles; tile += n_workers, ++tcount) {
-      int ft, tt;
-      tile_coords(tile, n_f, n_t, ft, tt);
-      const int f0 = ft * TILE_F + crank * 128, t0 = tt * BN;
+      const PTile pt = tile_at<BN>(p, ctrl, tile, n_f, n_t, grp);
+      const int f0 = pt.ft * TILE_F + crank * 128, t0 = pt.t0;
       const int f = f0 + lane_row;
       const int acc = tcount & 1;
       const uint32_t accph = (tcount >> 1) & 1;
@@ -405,6 +454,19 @@ umma_gemm_persistent_kernel(const __grid_constant__ CUtensorMap tmA,
           }
           fence_proxy_async_smem();
           epi_bar_sync();
+          if (p.n_groups > 0) {
+            // the rows behind the group belong to the next one: bounded 16-byte stores
+            __nv_bfloat16* out = static_cast<__nv_bfloat16*>(p.out);
+#pragma unroll
+            for (int u = 0; u < kChunkTok / 8; ++u) {
+              const int i = et + u * 128, r = i >> 4, fv = (i & 15) << 3;
+              const int t = t0 + c * kChunkTok + r;
+              if (ok && t < pt.t_end && f0 + fv < p.F)
+                *reinterpret_cast<uint4*>(out + (long long)t * p.ldo + f0 + fv) =
+                    *reinterpret_cast<const uint4*>(so + r * 128 + fv);
+            }
+            continue;
+          }
           if (et == 0 && ok && t0 + c * kChunkTok < p.T) {
             tma_store_2d(&tmOut, smem_u32(so), f0, t0 + c * kChunkTok);
             bulk_commit_group();
@@ -430,7 +492,7 @@ umma_gemm_persistent_kernel(const __grid_constant__ CUtensorMap tmA,
 #pragma unroll
             for (int b8 = 0; b8 < 4; ++b8)
               epilogue8<DUAL>(p, f, t0 + c + 8 * b8, v + 8 * b8, DUAL ? v2 + 8 * b8 : v2,
-                              p.T);
+                              pt.t_end);
           }
         }
       }
@@ -530,16 +592,17 @@ static int p_launch(E2hGemmParams& p, cudaStream_t stream) {
   CUtensorMap ta, ta2, tb, to, tr;
   int r;
   int mn3d = 0;
+  const long long a_rows = (long long)p.F * (p.n_groups > 0 ? p.n_groups : 1);
   if (p.a_mn_major && p.F % 64 == 0) {
     mn3d |= 1;
     r = p_map_mn3d(&ta, p.a, p.F, p.K, p.lda, 2);
   } else {
     r = p.a_mn_major ? p_map(&ta, p.a, p.F, p.K, p.lda, 64, 64, true)
-                     : p_map(&ta, p.a, p.K, p.F, p.lda, 64, 128, true);
+                     : p_map(&ta, p.a, p.K, a_rows, p.lda, 64, 128, true);
   }
   if (r) return r;
   if (DUAL) {
-    r = p_map(&ta2, p.a2, p.K, p.F, p.lda2, 64, 128, true);
+    r = p_map(&ta2, p.a2, p.K, a_rows, p.lda2, 64, 128, true);
     if (r) return r;
   } else {
     ta2 = ta;
@@ -554,6 +617,7 @@ static int p_launch(E2hGemmParams& p, cudaStream_t stream) {
   if (r) return r;
   int staged = (p.epi == E2H_EPI_STORE_BF16 || p.epi == E2H_EPI_RESIDUAL ||
                 (p.epi == E2H_EPI_SWIGLU && DUAL)) ? 1 : 0;
+  if (staged && p.n_groups > 0 && (p.F % 8)) staged = 0;
   if (staged && ((p.ldo % 8) || ((uintptr_t)p.out & 15))) staged = 0;
   if (staged && p.epi == E2H_EPI_RESIDUAL && ((uintptr_t)p.aux & 15)) staged = 0;
   if (!staged && p.epi == E2H_EPI_ROWMAJOR_BF16 && !p.accumulate && !DUAL && (p.ldo % 8) == 0 &&
@@ -602,7 +666,7 @@ static int p_launch(E2hGemmParams& p, cudaStream_t stream) {
   }
   if constexpr (PAIR) {
     // one cluster of two CTAs per 256 x 256 tile walker
-    const int n_tiles = (p.F / 256) * ((p.T + BN - 1) / BN);
+    const int n_tiles = (p.F / 256) * ((p.T + BN - 1) / BN + p.n_groups);
     const int pairs = n_tiles < n_sm / 2 ? n_tiles : n_sm / 2;
     cudaLaunchConfig_t cfg;
     memset(&cfg, 0, sizeof(cfg));
@@ -626,7 +690,7 @@ static int p_launch(E2hGemmParams& p, cudaStream_t stream) {
     cfg.numAttrs = na;
     return (int)cudaLaunchKernelEx(&cfg, kern, ta, ta2, tb, to, tr, p, staged, mn3d);
   }
-  const int n_tiles = ((p.F + 127) / 128) * ((p.T + BN - 1) / BN);
+  const int n_tiles = ((p.F + 127) / 128) * ((p.T + BN - 1) / BN + p.n_groups);
   const int grid = n_tiles < n_sm ? n_tiles : n_sm;
   return (int)launch(kern, dim3(grid), dim3(kPThreads), smem, stream, ta, ta2, tb, to, tr, p,
                      staged, mn3d);
@@ -640,7 +704,11 @@ extern "C" int e2h_gemm_persistent(const E2hGemmParams* pp, void* stream_v) {
   E2hGemmParams p = *pp;
   cudaStream_t stream = static_cast<cudaStream_t>(stream_v);
   if (p.F <= 0 || p.T <= 0 || p.K <= 0) return -1;
-  if (p.splitk > 1 || p.a_tiled || p.n_groups > 0 || p.tail_from) return -3;
+  if (p.splitk > 1 || p.a_tiled || p.tail_from) return -3;
+  if (p.n_groups > 0 &&
+      (p.n_groups > kPMaxGroups || p.a_mn_major || p.b_mn_major || p.group_off == nullptr ||
+       p.n_signal != 0 || (p.epi != E2H_EPI_STORE_BF16 && p.epi != E2H_EPI_SWIGLU)))
+    return -3;
   if (p.epi == E2H_EPI_RESIDUAL_F32 && p.aux != p.out) return -5;
   if (p.scale && (p.bias || p.act)) return -3;
   if ((p.bias || p.act) && p.epi != E2H_EPI_STORE_BF16 && p.epi != E2H_EPI_STORE_F32) return -3;

@@ -171,7 +171,11 @@ def gemm(a: torch.Tensor, b: torch.Tensor, *, epi: int, out: Optional[torch.Tens
                 splitk *= 2
         if kps <= 0:
             kps = 1 if (K % 64 or bn > 128) else 2
-        tf, persistent = 128, False
+        tf = 128
+        # many rows per group: persistent tiles walk group after group
+        persistent = n_groups <= 96 and T >= 128 * n_groups and group_tmax > 256
+        if persistent:
+            splitk, kps = 1, 1
     if (w8 or w4) and bn is None:
         bn = 64 if (T <= 64 or dual) else 128
     auto_tiles = (splitk is None and tf is None and kps <= 0 and th is None and not w8 and not w4

@@ -109,7 +109,8 @@ def test_packed_projection(dt, T, K, F, tail):
 @pytest.mark.parametrize("dt", DT)
 @pytest.mark.parametrize("n,E,top,K,F", [(1, 4, 2, 64, 40), (33, 5, 3, 88, 72), (64, 8, 8, 128, 128),
                                          (300, 3, 1, 96, 136), (700, 9, 4, 64, 64),
-                                         (5, 300, 6, 64, 64)])
+                                         (5, 300, 6, 64, 64), (900, 3, 2, 256, 192),
+                                         (400, 3, 2, 512, 264)])
 def test_routing_and_grouped_products(dt, n, E, top, K, F):
     from easy_to_hard_b200.ops import gemm, hybrid as hy
     dtype = DT[dt]
