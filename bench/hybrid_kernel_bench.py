@@ -120,9 +120,8 @@ def bovinex(size, batch, context, prompts, plen):
                         row("attention prep (norms, rotation, cache write)",
                             time_us(lambda: mix.prep(act, pos, slot)),
                             n * (2 * m.heads * m.dim * 2 + 2 * kv))
-                        both = time_us(lambda: mix.prompt(act, pos, slot, *seg))
-                        prep = time_us(lambda: mix.prep(act, pos, slot))
-                        row("attention (windowed flash, gate)", both - prep, io,
+                        row("attention (windowed flash, gate)", time_us(
+                            lambda: mix.attend(act, pos, slot, *seg)), io,
                             2.0 * vis * m.heads * (m.dim + m.vdim))
                 else:
                     st = m.heads * m.dim * m.vdim * 4

@@ -116,7 +116,12 @@ class WindowAttention:
     def prompt(self, act, pos, slot, seg, n_seg: int, seg_max: int) -> int:
         """Tokens seg[s] .. seg[s + 1] continue one sequence each. Returns the launches."""
         self.prep(act, pos, slot)
-        p = self.p
+        self.attend(act, pos, slot, seg, n_seg, seg_max)
+        return 2
+
+    def attend(self, act, pos, slot, seg, n_seg: int, seg_max: int) -> None:
+        """The second half of ``prompt``: attention and gate of tokens that are in the cache."""
+        p = self._bind(act, pos, slot)
         if (act.dtype == torch.bfloat16 and seg_max >= self.TENSOR_CORE_TOKENS
                 and p.dim % 8 == 0 and p.vdim % 8 == 0 and p.dim <= 128 and p.vdim <= 128):
             _lib.check(_lib.lib().e2h_flash_window(
@@ -125,7 +130,6 @@ class WindowAttention:
                 p.window, p.keep, p.status, _lib.stream()), "flash_window")
         else:
             self.from_cache(act, pos, slot)
-        return 2
 
     def from_cache(self, act, pos, slot) -> None:
         """Attention of tokens that ``prep`` has put into the cache."""
