@@ -2,8 +2,9 @@
 serves prompts, portions of prompts, single decode steps and mixtures of them.
 
 Tokens of all sequences lie one after the other (no padding); per-token positions and cache slots
-live on the device, so that the same captured decode step serves rows of unequal length. Per layer,
-with the parallel block (mixer and feed-forward read one norm):
+live on the device, so that the same captured decode step serves rows of unequal length. In a packed
+forward the longer pieces come first. Per layer, with the parallel block (mixer and feed-forward read
+one norm):
 
     norm of the fp32 residual            (first adds the expert outputs of the layer before)
     w_in GEMM: q, k, v, gate, activated up projection; fp32 tail: decay input, router logits
@@ -14,7 +15,17 @@ with the parallel block (mixer and feed-forward read one norm):
     w_out GEMM: residual += [gated heads, up] w_out^T
     experts: route + regroup, grouped SwiGLU GEMM, grouped down GEMM
 
-A decode step is 4 kernels per dense layer and 7 per expert layer.
+A decode step is 4 kernels per dense layer and 7 per expert layer. A sequential block (the feed-forward
+has a norm of its own) takes w_in without the feed-forward, then
+
+    norm of the residual
+    w_ff GEMM: activated up projection (dense, or the shared expert); fp32 tail: router logits
+    w_down GEMM: residual += up w_down^T
+    experts: route + regroup (rows weighted), grouped up GEMM + activation, grouped down GEMM
+
+and latent attention is three kernels in a decode step (queries absorb the key expansion; norm,
+rotation, cache write and attention over the latents; value expansion and gate), in prompts norm and
+rotation, the expansion of keys and values, and flash attention.
 """
 from __future__ import annotations
 
@@ -44,8 +55,9 @@ class _Scratch:
         self.x = torch.empty(n, cfg.dim, dtype=torch.float32, device=dev)
         self.h = buf(n, pad8(cfg.dim))
         self._act = torch.empty(n * max([b.f_main for b in blocks] or [8]), dtype=dt, device=dev)
-        self._tail = torch.empty(n * max([b.n_tail for b in blocks] + [8]), dtype=torch.float32,
-                                 device=dev)
+        self._ff = torch.empty(n * max([b.f_ff for b in blocks] or [8]), dtype=dt, device=dev)
+        self._tail = torch.empty(n * max([max(b.n_tail, b.n_ff_tail) for b in blocks] + [8]),
+                                 dtype=torch.float32, device=dev)
         moe = [b for b in blocks if b.layer.mlp is not None and b.layer.mlp.kind == "moe"]
         if moe:
             top = max(b.layer.mlp.top for b in moe)
@@ -62,8 +74,11 @@ class _Scratch:
     def act(self, n, cols):
         return self._act[: n * cols].view(n, cols)
 
+    def ff(self, n, cols):
+        return self._ff[: n * cols].view(n, cols)
+
     def tail(self, n, cols):
-        return self._tail[: n * cols].view(n, cols)
+        return self._tail[: n * cols].view(n, cols) if cols else None
 
     def ag(self, rows, cols):
         return self._ag[: rows * cols].view(rows, cols)
@@ -86,16 +101,31 @@ class HybridEngine(GenerationEngine):
         self.mixers = []
         for blk, store in zip(model.layers, self.cache.layers):
             m = blk.layer.mixer
-            offs = (blk.off_q, blk.off_k, blk.off_v, blk.off_g)
+            if m.kind == "gla":
+                self.mixers.append(hy.GatedLinearAttention(
+                    m, (blk.off_q, blk.off_k, blk.off_v, blk.off_g), store[0], blk.a2, blk.a2_b,
+                    blk.o_norm, self.eps))
+                continue
+            pairs = m.rot.dims // 2 if m.kind == "attention" else pad8(m.rot_dim) // 2
+            key = repr((m.rot, pairs))
+            if key not in tables:
+                tables[key] = m.rot.table(self.S, dev, pairs).contiguous()
             if m.kind == "attention":
-                key = repr(m.rot)
-                if key not in tables:
-                    tables[key] = m.rot.table(self.S, dev).contiguous()
-                self.mixers.append(hy.WindowAttention(m, offs, *store, tables[key], blk.q_norm,
-                                                      blk.k_norm, self.eps))
+                self.mixers.append(hy.WindowAttention(
+                    m, (blk.off_q, blk.off_k, blk.off_v, blk.off_g), *store, tables[key],
+                    blk.q_norm, blk.k_norm, self.eps))
             else:
-                self.mixers.append(hy.GatedLinearAttention(m, offs, store[0], blk.a2, blk.a2_b,
-                                                           blk.o_norm, self.eps))
+                self.mixers.append(hy.LatentAttention(
+                    m, (blk.off_q, blk.off_c, blk.off_g), store[0], tables[key], blk.w_kv,
+                    blk.w_uk_t, blk.c_norm, self.eps))
+        lat = [x for x in self.mixers if isinstance(x, hy.LatentAttention)]
+        self._latent = None
+        if lat:     # how prompt segments are served: widest window, whether keys are expanded
+            windows = [x.m.window for x in lat]
+            self._latent = (0 if 0 in windows else max(windows), all(x.can_expand for x in lat))
+            wide = max(x.p.H * x.rank for x in lat)
+            self._absorbed = [torch.empty(self.B * wide, dtype=model.dtype, device=dev)
+                              for _ in "qo"]
         self.slot = torch.zeros(self.B, dtype=torch.int32, device=dev)
         self.tok_pos = torch.zeros(self.B, dtype=torch.int32, device=dev)
         self.logits = torch.zeros(self.B, pad8(self.vocab), dtype=torch.float32, device=dev)
@@ -105,11 +135,12 @@ class HybridEngine(GenerationEngine):
         self.layer_trace: Optional[list] = None    # a list collects the residual after each layer
 
     # ------------------------------------------------------------------ forward
-    def _forward(self, w: _Scratch, n: int, tokens, pos, slot, *, seg=None, rows=None,
+    def _forward(self, w: _Scratch, n: int, tokens, pos, slot, *, seg=None, ctx=None, rows=None,
                  decode_counters: bool = False, hf=None, logits=None) -> None:
         """Runs ``n`` packed tokens through all layers. ``seg`` = (device offsets, segments,
-        longest segment), or None when every token is the next one of its own sequence. ``rows``
-        (int32, None: all) are the tokens whose ``logits`` are computed."""
+        longest segment), or None when every token is the next one of its own sequence; ``ctx``: the
+        segments' ``LatentContext``. ``rows`` (int32, None: all) are the tokens whose ``logits`` are
+        computed."""
         m, cfg = self.model, self.model.config
         W = cfg.dim
         x, h = w.x[:n], w.h[:n]
@@ -125,12 +156,19 @@ class HybridEngine(GenerationEngine):
                 self.layer_trace.append(x.clone())
             start, pending = {}, None
             act = w.act(n, blk.f_main)
-            tail = w.tail(n, blk.n_tail) if blk.n_tail else None
+            tail = w.tail(n, blk.n_tail)
             hw = h[:, :W]
+            dense = dict(act=blk.act) if blk.act else {}
             self._count(1 + gemm.linear_packed(
                 hw, blk.mat("w_in"), act, bias=blk.b_in, tail=tail,
-                act_from=blk.off_u if f is not None and f.kind == "dense" else None))
-            if blk.layer.mixer.kind == "attention":
+                **(dict(dense, act_from=blk.off_u) if cfg.parallel and dense else {})))
+            kind = blk.layer.mixer.kind
+            if kind == "latent":
+                if seg is None:
+                    self._count(mix.decode(act, pos, slot, *self._absorbed_rows(mix, n)))
+                else:
+                    self._count(mix.prompt(act, pos, slot, seg[0], ctx))
+            elif kind == "attention":
                 if seg is None:
                     mix.decode(act, pos, slot)
                     self._count(1)
@@ -143,6 +181,18 @@ class HybridEngine(GenerationEngine):
                 self._count(mix.prompt(act, tail, pos, slot, *seg))
             gemm.linear_residual_f32(act[:, blk.off_g:], blk.mat("w_out"), x)
             self._count(1)
+            if not cfg.parallel and f is not None:
+                hy.stream_norm(x, blk.norm2, h, eps=self.eps, offset=cfg.norm_offset)
+                tail = w.tail(n, blk.n_ff_tail)
+                self._count(1)
+                if dense:
+                    up = w.ff(n, blk.f_ff)
+                    self._count(1 + gemm.linear_packed(hw, blk.mat("w_ff"), up, bias=blk.b_ff,
+                                                       tail=tail, act_from=0, **dense))
+                    gemm.linear_residual_f32(up, blk.mat("w_down"), x)
+                else:
+                    gemm.linear_f32_out(hw, blk.mat("w_ff"), tail, bias=blk.b_ff)
+                    self._count(1)
             if f is not None and f.kind == "moe":
                 pending = self._experts(w, blk, n, hw, tail)
         if rows is None:
@@ -152,25 +202,43 @@ class HybridEngine(GenerationEngine):
         if rows_n:
             hy.stream_norm(x, m.norm, hf[:rows_n], eps=self.eps, offset=cfg.norm_offset,
                            experts=pending, rows=rows, **start)
-            gemm.linear_f32_out(hf[:rows_n, :W], m.head_w[:, :W], logits[:rows_n])
+            gemm.linear_f32_out(hf[:rows_n, :W], m.head_w[:, :W], logits[:rows_n],
+                                scale=cfg.logit_scale, softcap=cfg.logit_softcap)
             self._count(2)
         if self.layer_trace is not None:
             last = x.clone()
             if pending is not None and rows is not None:   # not yet added to the residual
                 y, place, ew = pending
-                last += (y.float()[place.long()][..., :W] * ew[..., None]).sum(1)
+                y = y.float()[place.long()][..., :W]
+                last += (y if ew is None else y * ew[..., None]).sum(1)
             self.layer_trace.append(last)
 
     def _experts(self, w: _Scratch, blk, n: int, hw, tail):
         f, W = blk.layer.mlp, self.model.config.dim
         place, ew = w.choice(n, f.top)
         k = hy.moe_route(tail[:, blk.off_r:], f.experts, f.top, hw, w.hg[: n * f.top, :W], w.off,
-                         place, ew, w.sel)
+                         place, ew, w.sel, score=f.score, weight_input=f.weight_input)
         hg, ag, y = w.hg[: n * f.top, :W], w.ag(n * f.top, blk.ffp), w.y[: n * f.top, :W]
-        gemm.grouped_swiglu(hg, blk.mat("e_gate"), blk.mat("e_up"), ag, w.off, f.experts, n)
+        if f.gated:
+            gemm.grouped_swiglu(hg, blk.mat("e_gate"), blk.mat("e_up"), ag, w.off, f.experts, n)
+        else:
+            gemm.grouped_linear(hg, blk.mat("e_up"), ag, w.off, f.experts, n, act=f.act)
         gemm.grouped_linear(ag, blk.mat("e_down"), y, w.off, f.experts, n)
         self._count(k + 2)
-        return y, place, ew
+        return y, place, None if f.weight_input else ew
+
+    def _absorbed_rows(self, mix, n: int):
+        """Absorbed queries and attended latents of ``n`` decode tokens."""
+        if n > self.B:
+            return ()
+        cols = mix.p.H * mix.rank
+        return (t[: n * cols].view(n, cols) for t in self._absorbed)
+
+    def _context(self, lengths, starts, slots) -> Optional[hy.LatentContext]:
+        if self._latent is None:
+            return None
+        window, expand = self._latent
+        return hy.LatentContext(lengths, starts, slots, window, expand, self.dev)
 
     # ------------------------------------------------------------------ steps over sequences
     def open(self, key: Hashable) -> None:
@@ -187,23 +255,29 @@ class HybridEngine(GenerationEngine):
         """Runs the next tokens of open sequences. ``entries``: (key, token ids, places among
         these tokens whose logits are wanted). Returns the wanted logits, fp32 [wanted, vocab], in
         the order of the entries and places."""
-        toks, pos, slot, seg, rows = [], [], [], [0], []
+        toks, pos, slot, seg = [], [], [], [0]
+        first: Dict[int, int] = {}       # entry -> its first packed token
+        starts, slots = [], []
         keys = [k for k, _, _ in entries]
         if len(set(keys)) != len(keys):
             raise ValueError("a sequence may appear once per step")
-        if len(toks) + sum(len(t) for _, t, _ in entries) > MAX_FORWARD_TOKENS:
+        if sum(len(t) for _, t, _ in entries) > MAX_FORWARD_TOKENS:
             return self._step_portions(entries)
-        for key, ids, want in entries:
+        for i in sorted(range(len(entries)), key=lambda i: -len(entries[i][1])):
+            key, ids, want = entries[i]
+            if any(not 0 <= int(j) < len(ids) for j in want):
+                raise ValueError("a wanted place lies outside the tokens of its entry")
             if not len(ids):
                 continue
             at = self.cache.extend(key, len(ids))
-            rows += [len(toks) + int(i) for i in want]
-            if any(not 0 <= int(i) < len(ids) for i in want):
-                raise ValueError("a wanted place lies outside the tokens of its entry")
+            first[i] = len(toks)
+            starts.append(at)
+            slots.append(self.cache.slot(key))
             toks += [int(t) for t in ids]
             pos += range(at, at + len(ids))
-            slot += [self.cache.slot(key)] * len(ids)
+            slot += [slots[-1]] * len(ids)
             seg.append(len(toks))
+        rows = [first[i] + int(j) for i, (_, _, want) in enumerate(entries) for j in want]
         n = len(toks)
         out = torch.empty(len(rows), self.vocab, dtype=torch.float32, device=self.dev)
         if n == 0:
@@ -216,8 +290,11 @@ class HybridEngine(GenerationEngine):
         w = self._scratch if n <= self.B else _Scratch(self.model, n)
         hf = torch.zeros(len(rows), pad8(self.cfg.dim), dtype=self.model.dtype, device=self.dev)
         logits = torch.empty(len(rows), pad8(self.vocab), dtype=torch.float32, device=self.dev)
+        alone = longest == 1
         self._forward(w, n, t_d, p_d, s_d, rows=rows_d,
-                      seg=None if longest == 1 else (seg_d, len(seg) - 1, longest),
+                      seg=None if alone else (seg_d, len(seg) - 1, longest),
+                      ctx=None if alone else self._context([b - a for a, b in zip(seg, seg[1:])],
+                                                           starts, slots),
                       hf=hf, logits=logits)
         out.copy_(logits[:, : self.vocab])
         return out
@@ -313,6 +390,7 @@ class HybridEngine(GenerationEngine):
 
     def _prefill_part(self, ids, T, pads, slots, pick):
         seg, cell, pos, slot, rows, fin = [0], [], [], [], [], []
+        pick = sorted(pick, key=lambda p: -p[2])
         for b, at, take in pick:
             lo = b * T + pads[b] + at
             cell += range(lo, lo + take)
@@ -329,9 +407,11 @@ class HybridEngine(GenerationEngine):
         tokens = ids.reshape(-1)[cell.long()]
         longest = max(t for _, _, t in pick)
         w = self._scratch if n <= self.B else _Scratch(self.model, n)
-        whole = len(fin) == ids.shape[0]
+        whole = fin == list(range(ids.shape[0]))
         logits = self.logits if whole else torch.empty_like(self.logits)
-        self._forward(w, n, tokens, pos, slot, seg=(seg_d, len(seg) - 1, longest), rows=rows_d,
-                      hf=self.hf, logits=logits)
+        ctx = self._context([t for _, _, t in pick], [a for _, a, _ in pick],
+                            [slots[b] for b, _, _ in pick])
+        self._forward(w, n, tokens, pos, slot, seg=(seg_d, len(seg) - 1, longest), ctx=ctx,
+                      rows=rows_d, hf=self.hf, logits=logits)
         if not whole and fin:
             self.logits[fin_d.long()] = logits[: len(fin)]

@@ -1,5 +1,6 @@
 """What live sequences keep between steps: a slot per sequence with, for every layer, the keys and
-values of its positions (attention) or its recurrent state (gated linear attention).
+values of its positions (attention), their latents and shared key parts (latent attention), or its
+recurrent state (gated linear attention).
 
 A slot is taken when a sequence opens and given back when it closes. Nothing is cleared in between:
 attention reads only positions the sequence has written, and the recurrent kernels start from zero
@@ -10,7 +11,7 @@ from typing import Dict, Hashable, List
 
 import torch
 
-from .hybrid import AttentionMixer, pad8
+from .hybrid import AttentionMixer, LatentMixer, pad8
 
 
 class SlotCache:
@@ -23,6 +24,9 @@ class SlotCache:
                 self.layers.append(tuple(
                     torch.zeros(slots, m.kv_heads, max_length, pad8(d), dtype=dtype,
                                 device=device) for d in (m.dim, m.vdim)))
+            elif isinstance(m, LatentMixer):
+                self.layers.append((torch.zeros(slots, max_length, pad8(m.kv_rank) + pad8(m.rot_dim),
+                                                dtype=dtype, device=device),))
             else:
                 self.layers.append((torch.zeros(slots, m.heads, m.dim, (m.vdim + 3) // 4 * 4,
                                                 dtype=torch.float32, device=device),))

@@ -49,6 +49,8 @@ class GemmParams(C.Structure):
         ("bias", C.c_void_p), ("act", C.c_int), ("act_from", C.c_int), ("tail_from", C.c_int),
         ("ldt", C.c_longlong), ("tail", C.c_void_p),
         ("n_groups", C.c_int), ("group_tmax", C.c_int), ("group_off", C.c_void_p),
+        ("out_scale", C.c_float), ("softcap", C.c_float),
+        ("n_batch", C.c_int), ("batch_k", C.c_int), ("batch_out", C.c_int),
     ]
 
 
@@ -80,6 +82,37 @@ class AttnWindowParams(C.Structure):
     ]
 
 
+class LatentParams(C.Structure):
+    """Mirror of ``LatentParams`` (csrc/latent_attn.cu)."""
+
+    _fields_ = [
+        ("act", C.c_void_p), ("ld", C.c_longlong), ("off_q", C.c_int), ("off_c", C.c_int),
+        ("ql", C.c_void_p), ("ol", C.c_void_p), ("cache", C.c_void_p), ("pos", C.c_void_p),
+        ("slot", C.c_void_p), ("n", C.c_int), ("slots", C.c_int), ("smax", C.c_int),
+        ("H", C.c_int), ("dim", C.c_int), ("rank", C.c_int), ("rot", C.c_int),
+        ("rank_n", C.c_int), ("rot_table", C.c_void_p), ("norm", C.c_void_p), ("eps", C.c_float),
+        ("scale", C.c_float), ("window", C.c_int), ("splits", C.c_int), ("ctx", C.c_void_p),
+        ("ctx_src", C.c_void_p), ("ctx_pos", C.c_void_p), ("ctx_slot", C.c_void_p),
+        ("n_ctx", C.c_int), ("n_long", C.c_int), ("status", C.c_void_p),
+    ]
+
+
+class FlashWindowArgs(C.Structure):
+    """Mirror of ``FlashWindowArgs`` (csrc/flash_window.cu)."""
+
+    _fields_ = [
+        ("act", C.c_void_p), ("ld", C.c_longlong), ("off_q", C.c_int), ("q_head", C.c_int),
+        ("off_g", C.c_int), ("k", C.c_void_p), ("ld_k", C.c_longlong), ("k_head", C.c_longlong),
+        ("k_slot", C.c_longlong), ("v", C.c_void_p), ("ld_v", C.c_longlong),
+        ("v_head", C.c_longlong), ("v_slot", C.c_longlong), ("k2", C.c_void_p),
+        ("ld_k2", C.c_longlong), ("rows", C.c_int), ("slots", C.c_int), ("smax", C.c_int),
+        ("shift", C.c_void_p), ("seg", C.c_void_p), ("n_seg", C.c_int), ("seg_max", C.c_int),
+        ("pos", C.c_void_p), ("slot", C.c_void_p), ("n", C.c_int), ("H", C.c_int), ("G", C.c_int),
+        ("dim", C.c_int), ("dim2", C.c_int), ("vdim", C.c_int), ("scale", C.c_float),
+        ("window", C.c_int), ("keep", C.c_int), ("status", C.c_void_p),
+    ]
+
+
 class GlaParams(C.Structure):
     """Mirror of ``E2hGlaParams`` (csrc/gla.cuh)."""
 
@@ -106,6 +139,7 @@ EPI_ROWMAJOR_F32_ACC = 5
 EPI_ROWMAJOR_BF16 = 6
 EPI_DUAL_STORE = 7
 EPI_RESIDUAL_F32 = 8
+EPI_GATE = 9
 
 _vp, _i, _ll, _f, _ull = C.c_void_p, C.c_int, C.c_longlong, C.c_float, C.c_ulonglong
 
@@ -119,13 +153,15 @@ _SIGNATURES = {
     "e2h_attn_prep": [C.POINTER(AttnWindowParams), _i, _vp],
     "e2h_attn_window": [C.POINTER(AttnWindowParams), _i, _i, _vp],
     "e2h_gla_chunk": [C.POINTER(GlaParams), _vp],
-    "e2h_flash_window": [_vp, _ll, _i, _i, _vp, _vp, _vp, _i, _i, _vp, _vp, _i, _i, _i, _i, _i, _i,
-                         _i, _i, _i, _f, _i, _i, _vp, _vp],
+    "e2h_flash_window": [C.POINTER(FlashWindowArgs), _vp],
+    "e2h_latent_prep": [C.POINTER(LatentParams), _i, _vp],
+    "e2h_latent_attn": [C.POINTER(LatentParams), _i, _i, _vp],
     "e2h_gla_step": [C.POINTER(GlaParams), _i, _vp],
     "e2h_gla_decay": [C.POINTER(GlaParams), _i, _vp],
     "e2h_gla_scan": [C.POINTER(GlaParams), _i, _vp],
     "e2h_gla_out": [C.POINTER(GlaParams), _i, _vp],
-    "e2h_moe_route": [_vp, _ll, _i, _i, _i, _vp, _ll, _i, _vp, _ll, _vp, _vp, _vp, _vp, _i, _vp],
+    "e2h_moe_route": [_vp, _ll, _i, _i, _i, _i, _i, _vp, _ll, _i, _vp, _ll, _vp, _vp, _vp, _vp, _i,
+                      _vp],
     "e2h_rmsnorm_fwd": [_vp, _vp, _vp, _i, C.POINTER(C.c_void_p), _i, _vp, _vp, _vp, _vp, _i, _i, _f,
                         _vp, _vp, _vp, _vp, _vp],
     "e2h_reduce_residual_norm_bf16": [_vp, C.POINTER(C.c_void_p), _i, _vp, _vp, _vp, _i, _i, _f,

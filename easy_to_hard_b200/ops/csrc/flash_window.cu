@@ -1,11 +1,19 @@
 // Prompt attention of the hybrid decoders on the tensor cores (bf16, head sizes up to 128): packed
 // sequences of unequal length, continued from the slot cache, a sliding window beside which the
 // first `keep` tokens stay visible, grouped queries, separate query/key and value sizes, sigmoid
-// output gate. attn_prep (attn_window.cu) has normed and rotated q in place and filled the cache.
+// output gate. attn_prep (attn_window.cu) or latent_prep (latent_attn.cu) has normed and rotated q in
+// place and filled the cache.
 //
-// One CTA = one (sequence, query head, 128-query block). Same roles and tensor-memory plan as the
-// causal kernel in flash_attn.cu: a TMA producer, a tcgen05 issuer, eight softmax warps (two
-// threads per query row), O accumulated in tensor memory with lazy rescaling. What differs:
+// Keys and values are rows of the slot cache, or of a buffer that holds, segment after segment, the
+// positions this forward looks at (keys and values expanded from latents): row = position + shift of
+// the segment. A key may have a second part of up to 64 columns that all heads share (the rotated
+// part of latent attention); it meets the columns of q behind the first part.
+//
+// One CTA = one (sequence, query head, 128-query block). Same roles as the causal kernel in
+// flash_attn.cu: a TMA producer, a tcgen05 issuer, eight softmax warps (two threads per query row),
+// O accumulated in tensor memory with lazy rescaling. What differs:
+//   * the probabilities go from registers into tensor memory and are the tensor-memory A operand of
+//     P V, so they take no shared memory and 192-wide keys fit with two stages;
 //   * the key tiles of a block are the tiles of the kept tokens followed by those from the window's
 //     lower edge to the diagonal; tiles in between are never loaded, and only tiles that an edge
 //     crosses test their keys;
@@ -38,6 +46,7 @@ constexpr float kWRescale = 8.f;
 struct FlashWindowParams {
   int H, G, n, slots, smax;
   int vdim;
+  const int* shift;            // [n_seg] key row - position, or null: rows of the slot cache
   float scale;
   int window, keep;            // window INT_MAX: unlimited
   const int* seg;              // [n_seg + 1]
@@ -57,13 +66,15 @@ struct FlashWindowCtrl {
   int abort_flag;
 };
 
-// KH / VH: 64-wide column blocks of the query/key and value heads.
-template <int KH, int VH>
+// KN / KR / VH: 64-wide column blocks of the query/key heads (own part, shared part) and of the values.
+template <int KN, int KR, int VH>
 __global__ void __launch_bounds__(kWThreads, 1)
-flash_window_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
+flash_window_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmQ2,
+                    const __grid_constant__ CUtensorMap tmK, const __grid_constant__ CUtensorMap tmK2,
                     const __grid_constant__ CUtensorMap tmV, const FlashWindowParams p) {
+  constexpr int KH = KN + KR;
   constexpr int kHalf = 128 * 128;               // [128 rows x 64] bf16
-  constexpr int kKT = KH * kHalf, kVT = VH * kHalf, kP = 2 * kHalf;
+  constexpr int kKT = KH * kHalf, kVT = VH * kHalf;
   constexpr int DV = VH * 64, DH = DV / 2;
   extern __shared__ __align__(1024) uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) &
@@ -73,9 +84,7 @@ flash_window_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
   uint8_t* q_s = smem + 2048;
   uint8_t* k_s = q_s + kKT;                      // 2 stages
   uint8_t* v_s = k_s + 2 * kKT;                  // 2 stages
-  uint8_t* p_s = v_s + 2 * kVT;                  // 2 buffers
 
-  pdl_launch_dependents();
   pdl_wait_prior();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int qb = gridDim.x - 1 - blockIdx.x, h = blockIdx.y, sg = blockIdx.z;
@@ -95,6 +104,8 @@ flash_window_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
   const int j_win = lo / kWK;
   const int n_kt = min((p.keep + kWK - 1) / kWK, j_win);  // tiles of kept tokens before it
   const int n_j = n_kt + p1 / kWK + 1 - j_win;
+  const int shift = p.shift ? p.shift[sg] : 0;   // key row = position + shift
+  const int kslot = p.shift ? 0 : slot;
   auto tile_key = [&](int it) { return (it < n_kt ? it : j_win + it - n_kt) * kWK; };
   volatile int* abort_flag = &ctrl->abort_flag;
 
@@ -116,16 +127,22 @@ flash_window_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
     tma_prefetch_desc(&tmQ);
     tma_prefetch_desc(&tmK);
     tma_prefetch_desc(&tmV);
+    if (KR) {
+      tma_prefetch_desc(&tmQ2);
+      tma_prefetch_desc(&tmK2);
+    }
   }
   if (warp == 1) {
-    tmem_alloc(smem_u32(&ctrl->tmem_base), 256);
+    tmem_alloc(smem_u32(&ctrl->tmem_base), 512);
     tmem_relinquish();
   }
   tc_fence_before();
   __syncthreads();
   tc_fence_after();
+  pdl_launch_dependents();      // with the tensor memory in hand: a dependent cannot take it first
   const uint32_t tmem_s = ctrl->tmem_base;
   const uint32_t tmem_o = tmem_s + 128;
+  const uint32_t tmem_p = tmem_s + 256;          // 2 buffers of 64 columns (128 bf16 per row)
 
   if (warp == 0 && lane == 0) {
     // ---------------- TMA producer ----------------
@@ -133,20 +150,24 @@ flash_window_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
     mbar_expect_tx(smem_u32(&ctrl->q_full), kKT);
 #pragma unroll
     for (int hf = 0; hf < KH; ++hf)
-      tma_load_4d(smem_u32(q_s + hf * kHalf), &tmQ, hf * 64, t_begin + q0, h, 0,
-                  smem_u32(&ctrl->q_full));
+      tma_load_4d(smem_u32(q_s + hf * kHalf), hf < KN ? &tmQ : &tmQ2, (hf < KN ? hf : hf - KN) * 64,
+                  t_begin + q0, h, 0, smem_u32(&ctrl->q_full));
     for (int it = 0; it < n_j; ++it) {
       const int s = it & 1;
       const uint32_t ph = (it >> 1) & 1;
-      const int key0 = tile_key(it);
+      const int key0 = tile_key(it) + shift;
       if (!mbar_wait(smem_u32(&ctrl->k_empty[s]), ph ^ 1, abort_flag, p.status,
                      kStatusTimeoutEmpty))
         break;
       mbar_expect_tx(smem_u32(&ctrl->k_full[s]), kKT);
 #pragma unroll
       for (int hf = 0; hf < KH; ++hf)
-        tma_load_4d(smem_u32(k_s + s * kKT + hf * kHalf), &tmK, hf * 64, key0, hk, slot,
-                    smem_u32(&ctrl->k_full[s]));
+        if (hf < KN)
+          tma_load_4d(smem_u32(k_s + s * kKT + hf * kHalf), &tmK, hf * 64, key0, hk, kslot,
+                      smem_u32(&ctrl->k_full[s]));
+        else
+          tma_load_4d(smem_u32(k_s + s * kKT + hf * kHalf), &tmK2, (hf - KN) * 64, key0, 0, kslot,
+                      smem_u32(&ctrl->k_full[s]));
       issued_k = it + 1;
       if (!mbar_wait(smem_u32(&ctrl->v_empty[s]), ph ^ 1, abort_flag, p.status,
                      kStatusTimeoutEmpty))
@@ -154,7 +175,7 @@ flash_window_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
       mbar_expect_tx(smem_u32(&ctrl->v_full[s]), kVT);
 #pragma unroll
       for (int hf = 0; hf < VH; ++hf)
-        tma_load_4d(smem_u32(v_s + s * kVT + hf * kHalf), &tmV, hf * 64, key0, hk, slot,
+        tma_load_4d(smem_u32(v_s + s * kVT + hf * kHalf), &tmV, hf * 64, key0, hk, kslot,
                     smem_u32(&ctrl->v_full[s]));
       issued_v = it + 1;
     }
@@ -206,12 +227,12 @@ flash_window_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
                      kStatusTimeoutFull);
       if (!ok) break;
       tc_fence_after();
-      const uint32_t pa = sw128_desc_lo(smem_u32(p_s + (it & 1) * kP), 16);
+      const uint32_t pa = tmem_p + (it & 1) * 64;
       const uint32_t va = sw128_desc_lo(smem_u32(v_s + s * kVT), kHalf);
 #pragma unroll
       for (int kk = 0; kk < kWK / 16; ++kk)
-        umma_f16_lohi(tmem_o, pa + (((kk / 4) * kHalf + (kk % 4) * 32) >> 4), d_hi,
-                      va + ((kk * 2048) >> 4), d_hi, idesc_o, (it > 0 || kk > 0) ? 1u : 0u);
+        umma_f16_ts(tmem_o, pa + kk * 8, va + ((kk * 2048) >> 4), d_hi, idesc_o,
+                    (it > 0 || kk > 0) ? 1u : 0u);
       umma_commit(smem_u32(&ctrl->v_empty[s]));
       umma_commit(smem_u32(&ctrl->p_empty[it & 1]));
       umma_commit(smem_u32(&ctrl->o_full));
@@ -294,24 +315,23 @@ flash_window_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
       if (ok) ok = mbar_wait(smem_u32(&ctrl->p_empty[it & 1]), ((it >> 1) & 1) ^ 1, abort_flag,
                              p.status, kStatusTimeoutEmpty);
       ok = __all_sync(0xffffffffu, ok);
-      uint8_t* prow = p_s + (it & 1) * kP + ch * kHalf + row * 128;
       float rs = 0.f;
+      tc_fence_after();
 #pragma unroll
-      for (int c8 = 0; c8 < 8; ++c8) {
-        uint32_t packed[4];
+      for (int q = 0; q < 2; ++q) {
+        uint32_t packed[16];
 #pragma unroll
-        for (int e = 0; e < 4; ++e) {
-          const float p0_ = ex2_approx(sv[c8 * 8 + 2 * e] - msafe);
-          const float p1_ = ex2_approx(sv[c8 * 8 + 2 * e + 1] - msafe);
+        for (int e = 0; e < 16; ++e) {
+          const float p0_ = ex2_approx(sv[32 * q + 2 * e] - msafe);
+          const float p1_ = ex2_approx(sv[32 * q + 2 * e + 1] - msafe);
           rs += p0_ + p1_;
           const __nv_bfloat162 pk = __floats2bfloat162_rn(p0_, p1_);
           packed[e] = *reinterpret_cast<const uint32_t*>(&pk);
         }
-        *reinterpret_cast<uint4*>(prow + ((c8 ^ (row & 7)) << 4)) =
-            make_uint4(packed[0], packed[1], packed[2], packed[3]);
+        if (ok) tmem_st_x16(tmem_p + (it & 1) * 64 + lane_off + ch * 32 + q * 16, packed);
       }
       l += rs;
-      fence_proxy_async_smem();
+      tmem_st_wait();
       tc_fence_before();
       __syncwarp();
       if (lane == 0) mbar_arrive(smem_u32(&ctrl->p_full));
@@ -360,66 +380,108 @@ flash_window_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
   }
   tc_fence_before();
   __syncthreads();
-  if (warp == 1) tmem_dealloc(ctrl->tmem_base, 256);
+  if (warp == 1) tmem_dealloc(ctrl->tmem_base, 512);
 }
 
-template <int KH, int VH>
-static int flash_window_launch(const CUtensorMap& tq, const CUtensorMap& tk, const CUtensorMap& tv,
-                               const FlashWindowParams& p, dim3 grid, cudaStream_t stream) {
-  const size_t smem = 1024 + 2048 + (size_t)(3 * KH + 2 * VH) * 128 * 128 + 2 * (2 * 128 * 128);
+struct FlashWindowMaps {
+  CUtensorMap q, q2, k, k2, v;
+};
+
+template <int KN, int KR, int VH>
+static int flash_window_launch(const FlashWindowMaps& m, const FlashWindowParams& p, dim3 grid,
+                               cudaStream_t stream) {
+  const size_t smem = 1024 + 2048 + (size_t)(3 * (KN + KR) + 2 * VH) * 128 * 128;
+  static_assert(1024 + 2048 + (3 * (KN + KR) + 2 * VH) * 128 * 128 <= 227 * 1024, "shared memory");
   static std::once_flag once;
   static cudaError_t err = cudaSuccess;
   std::call_once(once, [&] {
-    err = cudaFuncSetAttribute(flash_window_kernel<KH, VH>,
+    err = cudaFuncSetAttribute(flash_window_kernel<KN, KR, VH>,
                                cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
   });
   if (err != cudaSuccess) return (int)err;
-  return (int)launch(flash_window_kernel<KH, VH>, grid, dim3(kWThreads), smem, stream, tq, tk, tv,
-                     p);
+  return (int)launch(flash_window_kernel<KN, KR, VH>, grid, dim3(kWThreads), smem, stream, m.q,
+                     m.q2, m.k, m.k2, m.v, p);
 }
+
+struct FlashWindowArgs {
+  void* act;                   // bf16 [n, ld]
+  long long ld;
+  int off_q, q_head;           // column of head 0 of q (rotated), columns from head to head
+  int off_g;                   // gate columns (H x vdim)
+  const void* k;               // key rows: strides of rows, heads and slots, in elements
+  long long ld_k, k_head, k_slot;
+  const void* v;
+  long long ld_v, v_head, v_slot;
+  const void* k2;              // shared key part [rows, ld_k2] or null
+  long long ld_k2;
+  int rows, slots, smax;       // rows of a slot (or of the buffer), slots, positions of a sequence
+  const int* shift;            // [n_seg] key row - position: keys lie in a buffer; null: in the slots
+  const int* seg;              // [n_seg + 1]
+  int n_seg, seg_max;
+  const int* pos;
+  const int* slot;
+  int n, H, G;
+  int dim, dim2, vdim;         // own and shared part of a key, value
+  float scale;
+  int window, keep;
+  int* status;
+};
 
 }  // namespace e2h
 
-// act: packed activation [n, ld], q at off_q (normed and rotated), gate at off_g; caches
-// [slots, G, smax, dimp / vdimp]; segments of at most seg_max tokens.
-extern "C" int e2h_flash_window(void* act, long long ld, int off_q, int off_g, const void* kc,
-                                const void* vc, const int* seg, int n_seg, int seg_max,
-                                const int* pos, const int* slot, int n, int slots, int smax, int H,
-                                int G, int dim, int vdim, int dimp, int vdimp, float scale,
-                                int window, int keep, int* status, void* stream_v) {
+extern "C" int e2h_flash_window(const e2h::FlashWindowArgs* ap, void* stream_v) {
   using namespace e2h;
-  if (n <= 0 || n_seg <= 0 || n_seg > 65535 || seg_max <= 0 || G <= 0 || H % G || H > 65535)
+  const FlashWindowArgs& a = *ap;
+  if (a.n <= 0 || a.n_seg <= 0 || a.n_seg > 65535 || a.seg_max <= 0 || a.G <= 0 || a.H % a.G ||
+      a.H > 65535 || a.rows <= 0 || a.slots <= 0)
     return -1;
-  if (dim <= 0 || vdim <= 0 || dim > 128 || vdim > 128 || dim % 8 || vdim % 8 || dimp % 8 ||
-      vdimp % 8 || ld % 8 || off_q % 8 || off_g % 8)
+  if (a.dim <= 0 || a.vdim <= 0 || a.dim > 128 || a.vdim > 128 || a.dim2 < 0 || a.dim2 > 64 ||
+      (a.dim | a.dim2 | a.vdim | a.off_q | a.q_head | a.off_g) % 8 ||
+      (a.ld | a.ld_k | a.k_head | a.k_slot | a.ld_v | a.v_head | a.v_slot | a.ld_k2) % 8)
     return -2;
-  __nv_bfloat16* a = static_cast<__nv_bfloat16*>(act);
-  if ((reinterpret_cast<uintptr_t>(a) | reinterpret_cast<uintptr_t>(kc) |
-       reinterpret_cast<uintptr_t>(vc)) & 15)
+  if ((a.dim2 > 0) != (a.k2 != nullptr) || (a.k2 && !a.shift)) return -2;
+  __nv_bfloat16* act = static_cast<__nv_bfloat16*>(a.act);
+  if ((reinterpret_cast<uintptr_t>(act) | reinterpret_cast<uintptr_t>(a.k) |
+       reinterpret_cast<uintptr_t>(a.k2) | reinterpret_cast<uintptr_t>(a.v)) & 15)
     return -3;
-  CUtensorMap tq, tk, tv;
-  int r = make_map4d(&tq, a + off_q, dim, n, H, 1, (long long)n * ld, ld, dim, kWQ);
+  FlashWindowMaps m;
+  const long long all_q = (long long)a.n * a.ld;
+  int r = make_map4d(&m.q, act + a.off_q, a.dim, a.n, a.H, 1, all_q, a.ld, a.q_head, kWQ);
   if (r) return r;
-  r = make_map4d(&tk, kc, dim, smax, G, slots, (long long)G * smax * dimp, dimp,
-                 (long long)smax * dimp, kWK);
+  r = make_map4d(&m.k, a.k, a.dim, a.rows, a.G, a.slots, a.k_slot, a.ld_k, a.k_head, kWK);
   if (r) return r;
-  r = make_map4d(&tv, vc, vdim, smax, G, slots, (long long)G * smax * vdimp, vdimp,
-                 (long long)smax * vdimp, kWK);
+  r = make_map4d(&m.v, a.v, a.vdim, a.rows, a.G, a.slots, a.v_slot, a.ld_v, a.v_head, kWK);
   if (r) return r;
+  m.q2 = m.q;
+  m.k2 = m.k;
+  if (a.dim2) {
+    r = make_map4d(&m.q2, act + a.off_q + a.dim, a.dim2, a.n, a.H, 1, all_q, a.ld, a.q_head, kWQ);
+    if (r) return r;
+    const long long all_k = (long long)a.rows * a.ld_k2;
+    r = make_map4d(&m.k2, a.k2, a.dim2, a.rows, 1, 1, all_k, a.ld_k2, all_k, kWK);
+    if (r) return r;
+  }
   FlashWindowParams p;
-  p.H = H; p.G = G; p.n = n; p.slots = slots; p.smax = smax; p.vdim = vdim;
-  p.scale = scale;
-  p.window = window > 0 ? window : INT_MAX;
-  p.keep = keep;
-  p.seg = seg; p.pos = pos; p.slot = slot;
-  p.gate = a + off_g;
-  p.ld = ld;
-  p.status = status;
-  const dim3 grid((seg_max + kWQ - 1) / kWQ, H, n_seg);
+  p.H = a.H; p.G = a.G; p.n = a.n; p.slots = a.shift ? INT_MAX : a.slots; p.smax = a.smax;
+  p.vdim = a.vdim;
+  p.shift = a.shift;
+  p.scale = a.scale;
+  p.window = a.window > 0 ? a.window : INT_MAX;
+  p.keep = a.keep;
+  p.seg = a.seg; p.pos = a.pos; p.slot = a.slot;
+  p.gate = act + a.off_g;
+  p.ld = a.ld;
+  p.status = a.status;
+  const dim3 grid((a.seg_max + kWQ - 1) / kWQ, a.H, a.n_seg);
   cudaStream_t s = static_cast<cudaStream_t>(stream_v);
-  if (dim <= 64)
-    return vdim <= 64 ? flash_window_launch<1, 1>(tq, tk, tv, p, grid, s)
-                      : flash_window_launch<1, 2>(tq, tk, tv, p, grid, s);
-  return vdim <= 64 ? flash_window_launch<2, 1>(tq, tk, tv, p, grid, s)
-                    : flash_window_launch<2, 2>(tq, tk, tv, p, grid, s);
+#define E2H_FW(KN_, KR_)                                              \
+  return a.vdim <= 64 ? flash_window_launch<KN_, KR_, 1>(m, p, grid, s) \
+                      : flash_window_launch<KN_, KR_, 2>(m, p, grid, s)
+  if (a.dim2) {
+    if (a.dim <= 64) E2H_FW(1, 1);
+    E2H_FW(2, 1);
+  }
+  if (a.dim <= 64) E2H_FW(1, 0);
+  E2H_FW(2, 0);
+#undef E2H_FW
 }

@@ -21,12 +21,29 @@ __device__ __forceinline__ void bias_act(const E2hGemmParams& p, int f, float* v
 #pragma unroll
     for (int j = 0; j < N; ++j) v[j] += b;
   }
-  if (p.act == 1 && f >= p.act_from && (p.tail_from <= 0 || f < p.tail_from)) {
+  if (p.act && f >= p.act_from && (p.tail_from <= 0 || f < p.tail_from)) {
+    if (p.act == 1) {
 #pragma unroll
-    for (int j = 0; j < N; ++j) {
-      const float r = fmaxf(v[j], 0.f);
-      v[j] = r * r;
+      for (int j = 0; j < N; ++j) {
+        const float r = fmaxf(v[j], 0.f);
+        v[j] = r * r;
+      }
+    } else {
+#pragma unroll
+      for (int j = 0; j < N; ++j) v[j] = gelu_erf(v[j]);
     }
+  }
+}
+// Scale and soft cap of the fp32 store (logits).
+template <int N>
+__device__ __forceinline__ void scale_cap(const E2hGemmParams& p, float* v) {
+  if (p.out_scale != 0.f) {
+#pragma unroll
+    for (int j = 0; j < N; ++j) v[j] *= p.out_scale;
+  }
+  if (p.softcap != 0.f) {
+#pragma unroll
+    for (int j = 0; j < N; ++j) v[j] = p.softcap * tanhf(v[j] / p.softcap);
   }
 }
 __device__ __forceinline__ bool in_tail(const E2hGemmParams& p, int f) {
@@ -42,10 +59,11 @@ __device__ __forceinline__ void store_tail(const E2hGemmParams& p, int f, int t0
 }
 
 // Applies the epilogue to 8 consecutive token columns of one feature. Tokens from t_end on are
-// masked (p.T, or the end of the group in a grouped product).
+// masked (p.T, or the end of the group in a grouped product); o_col: first output column of this
+// matrix of a batched product.
 template <bool DUAL>
 __device__ __forceinline__ void epilogue8(const E2hGemmParams& p, int f, int t0, float* v,
-                                          float* v2, int t_end) {
+                                          float* v2, int t_end, int o_col = 0) {
   const bool f_ok = f < p.F;
   if (p.scale != nullptr) {
     const float s = f_ok ? p.scale[f] : 0.f;
@@ -69,17 +87,29 @@ __device__ __forceinline__ void epilogue8(const E2hGemmParams& p, int f, int t0,
 #pragma unroll
       for (int j = 0; j < 8; ++j) {
         const int t = t0 + j;
-        if (t < t_end) out[(long long)t * p.ldo + f] = __float2bfloat16_rn(v[j]);
+        if (t < t_end) out[(long long)t * p.ldo + o_col + f] = __float2bfloat16_rn(v[j]);
+      }
+    } break;
+    case E2H_EPI_GATE: {
+      __nv_bfloat16* out = static_cast<__nv_bfloat16*>(p.out);
+      if (!f_ok) break;
+#pragma unroll
+      for (int j = 0; j < 8; ++j) {
+        const int t = t0 + j;
+        if (t >= t_end) continue;
+        __nv_bfloat16* dst = out + (long long)t * p.ldo + o_col + f;
+        *dst = __float2bfloat16_rn(v[j] * sigmoid_fast(__bfloat162float(*dst)));
       }
     } break;
     case E2H_EPI_STORE_F32: {
       float* out = static_cast<float*>(p.out);
       if (!f_ok) break;
       bias_act<8>(p, f, v);
+      scale_cap<8>(p, v);
 #pragma unroll
       for (int j = 0; j < 8; ++j) {
         const int t = t0 + j;
-        if (t < t_end) out[(long long)t * p.ldo + f] = v[j];
+        if (t < t_end) out[(long long)t * p.ldo + o_col + f] = v[j];
       }
     } break;
     case E2H_EPI_RESIDUAL_F32: {
@@ -254,7 +284,7 @@ __device__ __forceinline__ void epilogue8(const E2hGemmParams& p, int f, int t0,
 // origins are 16-byte aligned.
 __host__ __device__ inline bool epi_can_stage(const E2hGemmParams& p, int tile_rows) {
   if (p.epi != E2H_EPI_STORE_BF16 && p.epi != E2H_EPI_RESIDUAL && p.epi != E2H_EPI_SWIGLU &&
-      p.epi != E2H_EPI_ROPE_KV)
+      p.epi != E2H_EPI_ROPE_KV && p.epi != E2H_EPI_GATE)
     return false;
   if ((p.F & 7) || (p.ldo & 7) || (tile_rows & 7) || (p.tail_from & 7)) return false;
   if (reinterpret_cast<uintptr_t>(p.out) & 15) return false;
@@ -371,7 +401,7 @@ __device__ __forceinline__ void stage8(const E2hGemmParams& p, int f, int t0, fl
 // thread's index among the epilogue threads, which have synchronised after stage8.
 __device__ __forceinline__ void flush_tile(const E2hGemmParams& p, const __nv_bfloat16* tile,
                                            int pitch, int f_first, int t_first, int n_tok,
-                                           int tid, int nthreads, int t_end) {
+                                           int tid, int nthreads, int t_end, int o_col = 0) {
   const int vpr = pitch >> 3;
   const int total = n_tok * vpr;
   __nv_bfloat16* out = static_cast<__nv_bfloat16*>(p.out);
@@ -382,8 +412,16 @@ __device__ __forceinline__ void flush_tile(const E2hGemmParams& p, const __nv_bf
     const int t = t_first + r, f = f_first + fv;
     if (t >= t_end || f >= p.F || in_tail(p, f)) continue;
     uint4 val = *reinterpret_cast<const uint4*>(tile + r * pitch + fv);
-    __nv_bfloat16* dst = out + (long long)t * p.ldo + f;
-    if (p.epi == E2H_EPI_RESIDUAL) {
+    __nv_bfloat16* dst = out + (long long)t * p.ldo + o_col + f;
+    if (p.epi == E2H_EPI_GATE) {
+      const uint4 gate = *reinterpret_cast<const uint4*>(dst);
+      const __nv_bfloat162* g = reinterpret_cast<const __nv_bfloat162*>(&gate);
+      __nv_bfloat162* o = reinterpret_cast<__nv_bfloat162*>(&val);
+#pragma unroll
+      for (int k = 0; k < 4; ++k)
+        o[k] = __floats2bfloat162_rn(__bfloat162float(o[k].x) * sigmoid_fast(__bfloat162float(g[k].x)),
+                                     __bfloat162float(o[k].y) * sigmoid_fast(__bfloat162float(g[k].y)));
+    } else if (p.epi == E2H_EPI_RESIDUAL) {
       const uint4 res = *reinterpret_cast<const uint4*>(
           static_cast<const __nv_bfloat16*>(p.aux) + (long long)t * p.ldo + f);
       const __nv_bfloat162* a = reinterpret_cast<const __nv_bfloat162*>(&val);

@@ -1,7 +1,8 @@
 // Linear layers in true 32-bit (FFMA, no reduced-precision tensor mode): the same parameter block
 // and conventions as e2h_gemm_umma with fp32 operands, for models that run in fp32. 64 x 64 tiles,
 // 256 threads with 4 x 4 outputs each. Epilogues: plain store, fp32 residual, SwiGLU on a dual
-// operand; bias, squared ReLU, the tail columns and grouped products as in gemm_umma.cu.
+// operand, sigmoid gate; bias, activations, the tail columns, grouped and batched products, scale and
+// soft cap as in gemm_umma.cu.
 #include <cuda_runtime.h>
 #include <stdint.h>
 
@@ -31,6 +32,15 @@ __global__ void __launch_bounds__(256) gemm_f32_kernel(const E2hGemmParams p) {
     if (t0 >= t_end || t0 < 0) return;
     a += (long long)g * p.F * p.lda;
     if (DUAL) a2 += (long long)g * p.F * p.lda2;
+  }
+  int o_col = 0;
+  if (p.n_batch > 0) {
+    const int per = (p.T + kF32Tile - 1) / kF32Tile;
+    const int g = blockIdx.y / per;
+    t0 = (blockIdx.y - g * per) * kF32Tile;
+    a += (long long)g * p.F * p.lda;
+    b += g * p.batch_k;
+    o_col = g * p.batch_out;
   }
   const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;   // features 4 tx.., tokens 4 ty..
   float acc[4][4], acc2[DUAL ? 4 : 1][4];
@@ -88,17 +98,24 @@ __global__ void __launch_bounds__(256) gemm_f32_kernel(const E2hGemmParams p) {
         v = v / (1.f + expf(-v)) * acc2[i][j];
       } else {
         if (p.bias) v += p.bias[f];
-        if (p.act == 1 && f >= p.act_from && (p.tail_from <= 0 || f < p.tail_from)) {
-          v = fmaxf(v, 0.f);
-          v *= v;
+        if (p.act && f >= p.act_from && (p.tail_from <= 0 || f < p.tail_from)) {
+          if (p.act == 1) {
+            v = fmaxf(v, 0.f);
+            v *= v;
+          } else {
+            v = gelu_erf(v);
+          }
         }
+        if (p.out_scale != 0.f) v *= p.out_scale;
+        if (p.softcap != 0.f) v = p.softcap * tanhf(v / p.softcap);
+        if (p.epi == E2H_EPI_GATE) v *= 1.f / (1.f + expf(-out[(long long)t * p.ldo + o_col + f]));
         if (p.epi == E2H_EPI_RESIDUAL_F32) v += res[(long long)t * p.ldo + f];
         if (p.tail_from > 0 && f >= p.tail_from) {
           p.tail[(long long)t * p.ldt + (f - p.tail_from)] = v;
           continue;
         }
       }
-      out[(long long)t * p.ldo + f] = v;
+      out[(long long)t * p.ldo + o_col + f] = v;
     }
   }
 }
@@ -108,13 +125,16 @@ __global__ void __launch_bounds__(256) gemm_f32_kernel(const E2hGemmParams p) {
 extern "C" int e2h_gemm_f32(const E2hGemmParams* p, void* stream) {
   using namespace e2h;
   if (p->F <= 0 || p->T <= 0 || p->K <= 0 || p->a_mn_major || p->b_mn_major || p->scale) return -1;
-  if (p->epi != E2H_EPI_STORE_F32 && p->epi != E2H_EPI_RESIDUAL_F32 && p->epi != E2H_EPI_SWIGLU)
+  if (p->epi != E2H_EPI_STORE_F32 && p->epi != E2H_EPI_RESIDUAL_F32 && p->epi != E2H_EPI_SWIGLU &&
+      p->epi != E2H_EPI_GATE)
     return -2;
+  if (p->n_batch > 0 && (p->n_groups > 0 || p->dual || p->tail_from || p->bias || p->act)) return -2;
   if ((p->epi == E2H_EPI_SWIGLU) != (p->dual != 0)) return -2;
   if (p->tail_from && (!p->tail || p->epi != E2H_EPI_STORE_F32)) return -2;
   if (p->n_groups > 0 && (!p->group_off || p->group_tmax <= 0)) return -2;
   const int tt = p->n_groups > 0 ? p->n_groups * ((p->group_tmax + kF32Tile - 1) / kF32Tile)
-                                 : (p->T + kF32Tile - 1) / kF32Tile;
+                                 : (p->n_batch > 0 ? p->n_batch : 1) *
+                                       ((p->T + kF32Tile - 1) / kF32Tile);
   if (tt > 65535) return -3;
   const dim3 grid((p->F + kF32Tile - 1) / kF32Tile, tt);
   if (p->dual)

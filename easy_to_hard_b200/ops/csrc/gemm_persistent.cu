@@ -709,6 +709,8 @@ extern "C" int e2h_gemm_persistent(const E2hGemmParams* pp, void* stream_v) {
       (p.n_groups > kPMaxGroups || p.a_mn_major || p.b_mn_major || p.group_off == nullptr ||
        p.n_signal != 0 || (p.epi != E2H_EPI_STORE_BF16 && p.epi != E2H_EPI_SWIGLU)))
     return -3;
+  if (p.n_batch > 0 || p.epi == E2H_EPI_GATE) return -5;
+  if ((p.out_scale != 0.f || p.softcap != 0.f) && p.epi != E2H_EPI_STORE_F32) return -5;
   if (p.epi == E2H_EPI_RESIDUAL_F32 && p.aux != p.out) return -5;
   if (p.scale && (p.bias || p.act)) return -3;
   if ((p.bias || p.act) && p.epi != E2H_EPI_STORE_BF16 && p.epi != E2H_EPI_STORE_F32) return -3;

@@ -119,6 +119,15 @@ umma_gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant_
     if (t_end > p.T) t_end = p.T;                // offsets come from device memory
     if (t0 >= t_end || t0 < 0) return;
   }
+  int b_col = 0, o_col = 0;                      // first columns of B and out (batched product)
+  if (p.n_batch > 0) {
+    const int per = (p.T + BN - 1) / BN;
+    const int g = blockIdx.y / per;
+    t0 = (blockIdx.y - g * per) * BN;
+    fa0 = g * p.F + f0;
+    b_col = g * p.batch_k;
+    o_col = g * p.batch_out;
+  }
 
   const int kb_total = (p.K + kTileK - 1) / kTileK;
   const int kb_begin = (int)((long long)rank * kb_total / S);
@@ -239,7 +248,7 @@ umma_gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant_
         }
         const uint32_t b_dst = a_dst + a_bytes * (DUAL ? 2 : 1);
         if (!p.b_mn_major) {
-          tma_load_2d(b_dst, &tmB, k0, t0, bar);
+          tma_load_2d(b_dst, &tmB, b_col + k0, t0, bar);
         } else {
 #pragma unroll
           for (int c = 0; c < BN / 64; ++c)
@@ -438,7 +447,7 @@ umma_gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant_
                        c + 8 * b, TH, lane_valid ? lane_row : -1, &rope, t_end);
         } else {
           epilogue8<DUAL>(p, f, t0 + c_begin + c + 8 * b, v + 8 * b, DUAL ? v2 + 8 * b : v2,
-                            t_end);
+                            t_end, o_col);
         }
       }
     }
@@ -448,7 +457,7 @@ umma_gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant_
     asm volatile("bar.sync 1, 256;" ::: "memory");   // the eight epilogue warps
     if (acc_ok)
       flush_tile(p, stile, TH, f0, t0 + rank * slice, slice, threadIdx.x - 64, 256,
-                 t_end);
+                 t_end, o_col);
   }
 
   if (warp == 2 && lane == 0) E2H_PHASE(p.phase_clock, 9);
@@ -548,7 +557,7 @@ static int launch(const E2hGemmParams& p, const CUtensorMap& ta, const CUtensorM
   cudaLaunchConfig_t cfg;
   memset(&cfg, 0, sizeof(cfg));
   const int t_tiles = p.n_groups > 0 ? p.n_groups * ((p.group_tmax + BN - 1) / BN)
-                                     : (p.T + BN - 1) / BN;
+                                     : (p.n_batch > 0 ? p.n_batch : 1) * ((p.T + BN - 1) / BN);
   if (t_tiles > 65535) return -13;
   cfg.gridDim = dim3((p.F + th - 1) / th, t_tiles, p.splitk);
   cfg.blockDim = dim3(kThreads, 1, 1);
@@ -591,9 +600,16 @@ extern "C" int e2h_gemm_umma(const E2hGemmParams* pp, void* stream_v) {
     return -5;
   if ((p.bias || p.act || p.tail_from) && p.epi != E2H_EPI_STORE_BF16 && p.epi != E2H_EPI_STORE_F32)
     return -5;
+  // (the columns of B past K of one matrix are those of the next: A's zero fill cancels them)
+  if (p.n_batch > 0 && (p.n_groups > 0 || p.dual || p.a_tiled || p.a_mn_major || p.b_mn_major ||
+                        p.n_signal != 0 || p.tail_from || p.bias || p.act || (p.batch_k % 8) ||
+                        (p.batch_out % 8) || (p.epi != E2H_EPI_STORE_BF16 && p.epi != E2H_EPI_GATE)))
+    return -5;
+  if ((p.out_scale != 0.f || p.softcap != 0.f) && p.epi != E2H_EPI_STORE_F32) return -5;
   if (p.epi == E2H_EPI_RESIDUAL_F32 && p.aux != p.out) return -5;
   if (p.tail_from && (p.epi != E2H_EPI_STORE_BF16 || p.tail == nullptr)) return -5;
-  const long long a_rows = (long long)p.F * (p.n_groups > 0 ? p.n_groups : 1);
+  const long long a_rows = (long long)p.F * (p.n_groups > 0 ? p.n_groups : p.n_batch > 0 ? p.n_batch : 1);
+  const long long b_cols = p.n_batch > 0 ? (long long)(p.n_batch - 1) * p.batch_k + p.K : p.K;
   if ((p.lda % 8) || (p.ldb % 8) || (p.dual && (p.lda2 % 8))) return -6;  // 16-byte strides for TMA
   if (((uintptr_t)p.a & 15) || ((uintptr_t)p.b & 15)) return -7;
   if (p.tf != 64 && p.tf != 128) p.tf = 128;
@@ -604,7 +620,7 @@ extern "C" int e2h_gemm_umma(const E2hGemmParams* pp, void* stream_v) {
   if (p.kps < 1) p.kps = 1;
   if (p.kps > 8) p.kps = 8;
   // several k-blocks per stage ride on 3-D boxes: K-major operands with K % 64 == 0 only
-  if (p.a_mn_major || p.b_mn_major || p.a_tiled || (p.K % 64) != 0) p.kps = 1;
+  if (p.a_mn_major || p.b_mn_major || p.a_tiled || p.n_batch > 0 || (p.K % 64) != 0) p.kps = 1;
   const int stage_bytes = p.kps * (p.th * 128 * (p.dual ? 2 : 1) + p.bn * 128);
   const int budget = 227 * 1024 - 2048 - xchg_bytes(p.bn, p.splitk, p.dual, p.tf);
   int max_stages = budget / stage_bytes;
@@ -652,7 +668,7 @@ extern "C" int e2h_gemm_umma(const E2hGemmParams* pp, void* stream_v) {
     ta2 = ta;
   }
   if (!p.b_mn_major)
-    r = make_map(&tb, p.b, p.K, p.T, p.ldb, p.bn);
+    r = make_map(&tb, p.b, b_cols, p.T, p.ldb, p.bn);
   else
     r = make_map(&tb, p.b, p.T, p.K, p.ldb, 64);
   if (r) return r;

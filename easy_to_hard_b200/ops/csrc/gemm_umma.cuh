@@ -18,6 +18,7 @@ enum E2hEpilogue : int {
   E2H_EPI_ROWMAJOR_BF16 = 6,     // out[f*ldo + t] = bf16(acc)
   E2H_EPI_DUAL_STORE = 7,   // dual A: out[t*ldo+f] = bf16(acc1), out2[t*ldo2+f] = bf16(acc2)
   E2H_EPI_RESIDUAL_F32 = 8, // out[t*ldo + f] += acc, aux == out           (fp32 residual stream)
+  E2H_EPI_GATE = 9,         // out[t*ldo + f] = acc * sigmoid(out[t*ldo + f])  (out holds the gate)
 };
 
 struct E2hGemmParams {
@@ -70,7 +71,8 @@ struct E2hGemmParams {
   unsigned long long* phase_clock;  // builds with E2H_PHASE_CLOCK only: 16 time stamps per CTA
   // several projections of one input in one launch (E2H_EPI_STORE_BF16 / _STORE_F32)
   const float* bias;     // optional per-feature bias added to acc (after `scale`)
-  int act;               // 1: squared ReLU on the features >= act_from (not on the tail)
+  int act;               // on the features >= act_from (not on the tail): 1 squared ReLU,
+                         // 2 GELU (the erf form)
   int act_from;
   int tail_from;         // > 0: features >= tail_from leave as fp32 in tail[t*ldt + f - tail_from]
   long long ldt;
@@ -80,6 +82,12 @@ struct E2hGemmParams {
   int n_groups;
   int group_tmax;        // host bound of the rows of one group (sizes the grid)
   const int* group_off;  // device, n_groups + 1 ascending entries
+  // E2H_EPI_STORE_F32: acc * out_scale (0: as it is), then softcap * tanh(. / softcap) (0: as it is)
+  float out_scale, softcap;
+  // batched products (one matrix per head): A holds n_batch matrices of F rows one below the other;
+  // matrix g multiplies the columns g * batch_k .. + K of every row of B and fills the columns
+  // g * batch_out .. + F of every row of out
+  int n_batch, batch_k, batch_out;
 };
 
 #ifdef __cplusplus

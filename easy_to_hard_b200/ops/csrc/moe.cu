@@ -1,6 +1,8 @@
-// Mixture-of-experts routing: top-k of the fp32 router logits, softmax over the chosen ones, and
-// the regrouping of the tokens by expert for the grouped GEMMs (rows of expert e are
-// off[e] .. off[e + 1] of the regrouped activation, in token order, so nothing depends on timing).
+// Mixture-of-experts routing: top-k of the fp32 router logits, their weights (softmax over the chosen
+// ones, or the sigmoid of each), and the regrouping of the tokens by expert for the grouped GEMMs
+// (rows of expert e are off[e] .. off[e + 1] of the regrouped activation, in token order, so nothing
+// depends on timing). The regrouped rows may carry their weight (designs that weight the expert's
+// input instead of its output).
 //
 //   moe_route_small   one launch for a decode-sized batch: every CTA (one token) routes the whole
 //                     batch redundantly from its few logits and copies its own token's rows
@@ -20,9 +22,12 @@ constexpr int kMoeMaxTop = 16;
 constexpr int kMoeMaxExperts = 1024;
 constexpr int kMoeSmall = 1024;      // token * top bound of the one-launch form
 
-// One warp: the `top` largest of z[0..E) (ties: lower index), and their softmax. Every lane
-// returns with the whole result in idx / val (val holds the weights).
-__device__ __forceinline__ void warp_topk(const float* z, int E, int top, int* idx, float* val) {
+enum : int { kScoreSoftmax = 0, kScoreSigmoid = 1 };
+
+// One warp: the `top` largest of z[0..E) (ties: lower index), and their weights: softmax over them or
+// the sigmoid of each. Every lane returns with the whole result in idx / val (val holds the weights).
+__device__ __forceinline__ void warp_topk(const float* z, int E, int top, int score, int* idx,
+                                          float* val) {
   const int lane = threadIdx.x & 31;
   float last = INFINITY;
   int last_i = -1;
@@ -53,14 +58,31 @@ __device__ __forceinline__ void warp_topk(const float* z, int E, int top, int* i
     last_i = bi;
     if (j == 0) mx = bv;
     idx[j] = bi;
-    val[j] = expf(bv - mx);
+    val[j] = score == kScoreSigmoid ? sigmoid_f(bv) : expf(bv - mx);
     sum += val[j];
   }
-  for (int j = 0; j < top; ++j) val[j] /= sum;
+  if (score != kScoreSigmoid)
+    for (int j = 0; j < top; ++j) val[j] /= sum;
 }
 
+// dst = src * f (f == 1: a plain copy)
 template <typename T>
-__device__ __forceinline__ void copy_row(T* dst, const T* src, int W) {
+__device__ __forceinline__ void copy_row(T* dst, const T* src, int W, float f = 1.f) {
+  if (f != 1.f) {
+    if (W % 4 == 0 && ((reinterpret_cast<uintptr_t>(dst) | reinterpret_cast<uintptr_t>(src)) &
+                       (4 * sizeof(T) - 1)) == 0) {
+      for (int i = threadIdx.x * 4; i < W; i += blockDim.x * 4) {
+        float v[4];
+        load4(src + i, v);
+#pragma unroll
+        for (int k = 0; k < 4; ++k) v[k] *= f;
+        store4(dst + i, v);
+      }
+    } else {
+      for (int i = threadIdx.x; i < W; i += blockDim.x) dst[i] = from_f<T>(to_f(src[i]) * f);
+    }
+    return;
+  }
   if ((W * sizeof(T)) % 16 == 0 && ((reinterpret_cast<uintptr_t>(dst) |
                                      reinterpret_cast<uintptr_t>(src)) & 15) == 0) {
     const int n = W * sizeof(T) / 16;
@@ -76,11 +98,13 @@ constexpr int kRouteLogits = 8192;   // logits staged in shared memory
 
 template <typename T>
 __global__ void __launch_bounds__(kRouteThreads)
-moe_route_small_kernel(const float* z, long long ldz, int n, int E, int top, const T* h,
-                       long long ldh, int W, T* hg, long long ldg, int* off, int* place, float* w) {
+moe_route_small_kernel(const float* z, long long ldz, int n, int E, int top, int score, int scale_in,
+                       const T* h, long long ldh, int W, T* hg, long long ldg, int* off, int* place,
+                       float* w) {
   __shared__ int sel[kMoeSmall];
   __shared__ int count[kMoeMaxExperts];
   __shared__ int my_off[kMoeMaxTop], my_before[kMoeMaxTop];
+  __shared__ float my_w[kMoeMaxTop];
   extern __shared__ float z_s[];
   pdl_launch_dependents();
   pdl_wait_prior();
@@ -94,11 +118,11 @@ moe_route_small_kernel(const float* z, long long ldz, int n, int E, int top, con
   for (int t = warp; t < n; t += blockDim.x >> 5) {
     int idx[kMoeMaxTop];
     float val[kMoeMaxTop];
-    warp_topk(staged ? z_s + t * E : z + t * ldz, E, top, idx, val);
+    warp_topk(staged ? z_s + t * E : z + t * ldz, E, top, score, idx, val);
     if (lane == 0) {
       for (int j = 0; j < top; ++j) {
         sel[t * top + j] = idx[j];
-        if (t == t_me) w[t * top + j] = val[j];
+        if (t == t_me) w[t * top + j] = my_w[j] = val[j];
       }
     }
   }
@@ -116,7 +140,7 @@ moe_route_small_kernel(const float* z, long long ldz, int n, int E, int top, con
   for (int j = 0; j < top; ++j) {
     const int at = my_off[j] + my_before[j];
     if (threadIdx.x == 0) place[t_me * top + j] = at;
-    copy_row(hg + at * ldg, h + t_me * ldh, W);
+    copy_row(hg + at * ldg, h + t_me * ldh, W, scale_in ? my_w[j] : 1.f);
   }
   if (t_me == 0 && warp == 0) {
     int run = 0;
@@ -135,15 +159,15 @@ moe_route_small_kernel(const float* z, long long ldz, int n, int E, int top, con
   }
 }
 
-__global__ void moe_topk_kernel(const float* z, long long ldz, int n, int E, int top, int* sel,
-                                float* w) {
+__global__ void moe_topk_kernel(const float* z, long long ldz, int n, int E, int top, int score,
+                                int* sel, float* w) {
   pdl_launch_dependents();
   pdl_wait_prior();
   const int t = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
   if (t >= n) return;
   int idx[kMoeMaxTop];
   float val[kMoeMaxTop];
-  warp_topk(z + t * ldz, E, top, idx, val);
+  warp_topk(z + t * ldz, E, top, score, idx, val);
   if ((threadIdx.x & 31) == 0)
     for (int j = 0; j < top; ++j) {
       sel[t * top + j] = idx[j];
@@ -200,44 +224,48 @@ moe_group_kernel(const int* sel, int m, int E, int* off, int* place) {
 
 template <typename T>
 __global__ void moe_gather_kernel(const T* h, long long ldh, int W, int top, const int* place,
-                                  int rows, T* hg, long long ldg) {
+                                  const float* w, int rows, T* hg, long long ldg) {
   pdl_launch_dependents();
   pdl_wait_prior();
   const int t = blockIdx.x;
   for (int j = 0; j < top; ++j) {
     const int at = place[t * top + j];
-    if (at >= 0 && at < rows) copy_row(hg + at * ldg, h + t * ldh, W);
+    if (at >= 0 && at < rows)
+      copy_row(hg + at * ldg, h + t * ldh, W, w ? w[(long long)t * top + j] : 1.f);
   }
 }
 
 template <typename T>
-static int route(const float* z, long long ldz, int n, int E, int top, const void* h, long long ldh,
-                 int W, void* hg, long long ldg, int* off, int* place, float* w, int* sel,
-                 cudaStream_t s) {
+static int route(const float* z, long long ldz, int n, int E, int top, int score, int scale_in,
+                 const void* h, long long ldh, int W, void* hg, long long ldg, int* off, int* place,
+                 float* w, int* sel, cudaStream_t s) {
   if (n * top <= kMoeSmall && n <= 256)
     return (int)launch(moe_route_small_kernel<T>, dim3(n), dim3(kRouteThreads),
-                       n * E <= kRouteLogits ? (size_t)n * E * 4 : 0, s, z, ldz, n, E, top,
-                       static_cast<const T*>(h), ldh, W, static_cast<T*>(hg), ldg, off, place, w);
-  int r = (int)launch(moe_topk_kernel, dim3((n + 7) / 8), dim3(256), 0, s, z, ldz, n, E, top, sel, w);
+                       n * E <= kRouteLogits ? (size_t)n * E * 4 : 0, s, z, ldz, n, E, top, score,
+                       scale_in, static_cast<const T*>(h), ldh, W, static_cast<T*>(hg), ldg, off, place, w);
+  int r = (int)launch(moe_topk_kernel, dim3((n + 7) / 8), dim3(256), 0, s, z, ldz, n, E, top,
+                      score, sel, w);
   if (r) return r;
   r = (int)launch(moe_group_kernel, dim3(E), dim3(1024), 0, s, sel, n * top, E, off, place);
   if (r) return r;
   return (int)launch(moe_gather_kernel<T>, dim3(n), dim3(256), 0, s, static_cast<const T*>(h), ldh,
-                     W, top, place, n * top, static_cast<T*>(hg), ldg);
+                     W, top, place, scale_in ? w : nullptr, n * top, static_cast<T*>(hg), ldg);
 }
 
 }  // namespace e2h
 
 // z fp32 [n, ldz] router logits (bias included); h [n, ldh]; hg [n * top, ldg]; off int [E + 1];
-// place, w, sel [n, top].
-extern "C" int e2h_moe_route(const float* z, long long ldz, int n, int E, int top, const void* h,
-                             long long ldh, int W, void* hg, long long ldg, int* off, int* place,
-                             float* w, int* sel, int is_bf16, void* stream) {
+// place, w, sel [n, top]. score: 0 softmax over the chosen, 1 sigmoid; scale_in: the rows of hg carry
+// their weight.
+extern "C" int e2h_moe_route(const float* z, long long ldz, int n, int E, int top, int score,
+                             int scale_in, const void* h, long long ldh, int W, void* hg,
+                             long long ldg, int* off, int* place, float* w, int* sel, int is_bf16,
+                             void* stream) {
   using namespace e2h;
   if (n <= 0 || E <= 0 || E > kMoeMaxExperts || top <= 0 || top > kMoeMaxTop || top > E) return -1;
   if ((long long)n * top > 0x3fffffff) return -1;
-  return is_bf16 ? route<__nv_bfloat16>(z, ldz, n, E, top, h, ldh, W, hg, ldg, off, place, w, sel,
-                                        (cudaStream_t)stream)
-                 : route<float>(z, ldz, n, E, top, h, ldh, W, hg, ldg, off, place, w, sel,
-                                (cudaStream_t)stream);
+  return is_bf16 ? route<__nv_bfloat16>(z, ldz, n, E, top, score, scale_in, h, ldh, W, hg, ldg, off,
+                                        place, w, sel, (cudaStream_t)stream)
+                 : route<float>(z, ldz, n, E, top, score, scale_in, h, ldh, W, hg, ldg, off, place, w,
+                                sel, (cudaStream_t)stream);
 }

@@ -33,7 +33,7 @@ struct StreamNormParams {
   const void* y;            // T [n * top, ldy] expert outputs or null
   long long ldy;
   const int* place;         // [n, top] row of y
-  const float* ew;          // [n, top] weights
+  const float* ew;          // [n, top] weights or null (the outputs are weighted already)
   int top, y_rows;
   const int* rows;          // [n] or null
   int x_rows;
@@ -94,7 +94,7 @@ __global__ void stream_norm_kernel(const StreamNormParams p) {
         for (int j = 0; j < p.top; ++j) {
           int at = p.place[(long long)r * p.top + j];
           at = min(max(at, 0), p.y_rows - 1);
-          const float w = p.ew[(long long)r * p.top + j];
+          const float w = p.ew ? p.ew[(long long)r * p.top + j] : 1.f;
           float u[4];
           load4(static_cast<const T*>(p.y) + at * p.ldy + c, u);
 #pragma unroll
@@ -116,7 +116,8 @@ __global__ void stream_norm_kernel(const StreamNormParams p) {
         for (int j = 0; j < p.top; ++j) {
           int at = p.place[(long long)r * p.top + j];
           at = min(max(at, 0), p.y_rows - 1);
-          s += p.ew[(long long)r * p.top + j] * to_f(static_cast<const T*>(p.y)[at * p.ldy + c]);
+          s += (p.ew ? p.ew[(long long)r * p.top + j] : 1.f) *
+               to_f(static_cast<const T*>(p.y)[at * p.ldy + c]);
         }
         v += s;
       }
@@ -164,7 +165,7 @@ static int stream_norm_launch(const StreamNormParams& p, int n, cudaStream_t str
 
 extern "C" int e2h_stream_norm(const e2h::StreamNormParams* p, int n, int is_bf16, void* stream) {
   if (n <= 0 || p->W <= 0 || !p->x || !p->status) return -1;
-  if (p->y && (!p->place || !p->ew || p->top <= 0 || p->y_rows <= 0)) return -1;
+  if (p->y && (!p->place || p->top <= 0 || p->y_rows <= 0)) return -1;
   return is_bf16 ? e2h::stream_norm_launch<__nv_bfloat16>(*p, n, (cudaStream_t)stream)
                  : e2h::stream_norm_launch<float>(*p, n, (cudaStream_t)stream);
 }

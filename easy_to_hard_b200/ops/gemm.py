@@ -14,7 +14,7 @@ from typing import Optional
 import torch
 
 from . import _lib
-from ._lib import (EPI_DUAL_STORE, EPI_RESIDUAL, EPI_RESIDUAL_F32, EPI_ROPE_KV,
+from ._lib import (EPI_DUAL_STORE, EPI_GATE, EPI_RESIDUAL, EPI_RESIDUAL_F32, EPI_ROPE_KV,
                    EPI_ROWMAJOR_BF16, EPI_ROWMAJOR_F32_ACC, EPI_STORE_BF16, EPI_STORE_F32,
                    EPI_SWIGLU, GemmParams)
 
@@ -113,12 +113,16 @@ def gemm(a: torch.Tensor, b: torch.Tensor, *, epi: int, out: Optional[torch.Tens
          th: Optional[int] = None, bias: Optional[torch.Tensor] = None,
          act_from: Optional[int] = None, tail: Optional[torch.Tensor] = None,
          tail_from: int = 0, group_off: Optional[torch.Tensor] = None, n_groups: int = 0,
-         group_tmax: int = 0) -> None:
-    """Raw launch. ``bias`` (fp32 [F]), ``act_from`` (squared ReLU on the features from there
+         group_tmax: int = 0, act: str = "relu2", out_scale: float = 1.0, softcap: float = 0.0,
+         batch: Optional[tuple] = None) -> None:
+    """Raw launch. ``bias`` (fp32 [F]), ``act_from`` (activation ``act`` on the features from there
     on), ``tail`` / ``tail_from`` (the features from there on leave as fp32) belong to the plain
-    stores; ``group_off`` (int32 [n_groups + 1], ascending) makes the product grouped: ``a`` holds
+    stores, ``out_scale`` / ``softcap`` (cap * tanh(x * scale / cap)) to the fp32 one;
+    ``batch`` = (matrices, column step of b, column step of out): see ``batched_linear``;
+    ``group_off`` (int32 [n_groups + 1], ascending) makes the product grouped: ``a`` holds
     ``n_groups`` matrices below one another and rows group_off[g] .. group_off[g + 1] of ``b`` are
-    multiplied by matrix g (at most ``group_tmax`` rows each). Shapes: a is [F, K] (or [K, F] when a_mn_major), b is [T, K] (or [K, T]).
+    multiplied by matrix g (at most ``group_tmax`` rows each). Shapes: a is [F, K] (or [K, F] when
+    a_mn_major), b is [T, K] (or [K, T]).
     An int8 ``a`` (weight-only quantisation; ``scale`` holds the per-feature scales) streams as
     int8 through the converting kernel for up to 128 tokens and is expanded to a scratch bf16
     matrix first for larger token counts."""
@@ -176,10 +180,19 @@ def gemm(a: torch.Tensor, b: torch.Tensor, *, epi: int, out: Optional[torch.Tens
         persistent = n_groups <= 96 and T >= 128 * n_groups and group_tmax > 256
         if persistent:
             splitk, kps = 1, 1
+    if batch is not None:
+        assert F % batch[0] == 0 and not w8 and not w4 and not n_groups
+        F //= batch[0]
+        bn = bn or (64 if T <= 64 else 128 if T <= 128 else 256)
+        splitk, ctas = 1, -(-F // 128) * batch[0] * -(-T // bn)
+        while (splitk < 8 and ctas * splitk * 2 <= N_SM and -(-K // 64) // (splitk * 2) >= 2
+               and bn % (splitk * 2 * 8) == 0):
+            splitk *= 2
+        tf, kps, persistent = 128, 1, False
     if (w8 or w4) and bn is None:
         bn = 64 if (T <= 64 or dual) else 128
     auto_tiles = (splitk is None and tf is None and kps <= 0 and th is None and not w8 and not w4
-                  and not n_groups
+                  and not n_groups and batch is None
                   and not a_mn_major and not b_mn_major and tiled_shape is None
                   and K % 64 == 0 and STREAM_TILES)
     bn, splitk, stages, tf, kps = pick_tiles(F, T, K, dual, splitk, bn, stages, tf, kps)
@@ -250,9 +263,10 @@ def gemm(a: torch.Tensor, b: torch.Tensor, *, epi: int, out: Optional[torch.Tens
         assert bias.dtype == torch.float32 and bias.numel() >= F
         p.bias = bias.data_ptr()
     if act_from is not None:
-        p.act, p.act_from = 1, act_from
+        p.act, p.act_from = ACTIVATIONS[act], act_from
     if tail_from:
         p.tail_from, p.tail, p.ldt = tail_from, tail.data_ptr(), tail.stride(0)
+    _scale_and_batch(p, out_scale, softcap, batch)
     if n_groups:
         assert group_off.dtype == torch.int32 and group_off.numel() > n_groups
         p.n_groups, p.group_tmax, p.group_off = n_groups, group_tmax, group_off.data_ptr()
@@ -275,6 +289,19 @@ def gemm(a: torch.Tensor, b: torch.Tensor, *, epi: int, out: Optional[torch.Tens
                    "e2h_gemm_persistent")
     else:
         _lib.check(_lib.lib().e2h_gemm_umma(C.byref(p), _lib.stream()), "e2h_gemm_umma")
+
+
+# activation codes of the plain stores (bias_act in csrc/gemm_epilogue.cuh)
+ACTIVATIONS = {"relu2": 1, "gelu": 2}
+
+
+def _scale_and_batch(p: GemmParams, out_scale: float, softcap: float, batch) -> None:
+    if out_scale != 1.0:
+        assert out_scale
+        p.out_scale = out_scale
+    p.softcap = softcap
+    if batch is not None:
+        p.n_batch, p.batch_k, p.batch_out = batch
 
 
 class Int4Weight:
@@ -448,10 +475,13 @@ def linear_wgrad(dy: torch.Tensor, x: torch.Tensor, out: Optional[torch.Tensor] 
 # true 32-bit kernel (csrc/gemm_f32.cu). The residual stream and the tails are fp32 in both.
 
 def _gemm_f32(a, b, *, epi, out, a2=None, aux=None, bias=None, act_from=None, tail=None,
-              tail_from=0, group_off=None, n_groups=0, group_tmax=0) -> None:
+              tail_from=0, group_off=None, n_groups=0, group_tmax=0, act="relu2", out_scale=1.0,
+              softcap=0.0, batch=None) -> None:
     assert a.dtype == b.dtype == torch.float32 and a.shape[1] == b.shape[1]
     p = GemmParams()
-    p.F, p.T, p.K = a.shape[0] // max(n_groups, 1), b.shape[0], a.shape[1]
+    p.F = a.shape[0] // max(n_groups, batch[0] if batch else 1, 1)
+    p.T, p.K = b.shape[0], a.shape[1]
+    _scale_and_batch(p, out_scale, softcap, batch)
     p.epi, p.lda, p.ldb, p.a, p.b = epi, _ld(a), _ld(b), a.data_ptr(), b.data_ptr()
     if a2 is not None:
         p.dual, p.a2, p.lda2 = 1, a2.data_ptr(), _ld(a2)
@@ -462,7 +492,7 @@ def _gemm_f32(a, b, *, epi, out, a2=None, aux=None, bias=None, act_from=None, ta
     if bias is not None:
         p.bias = bias.data_ptr()
     if act_from is not None:
-        p.act, p.act_from = 1, act_from
+        p.act, p.act_from = ACTIVATIONS[act], act_from
     if tail_from:
         p.tail_from, p.tail, p.ldt = tail_from, tail.data_ptr(), tail.stride(0)
     if n_groups:
@@ -470,20 +500,20 @@ def _gemm_f32(a, b, *, epi, out, a2=None, aux=None, bias=None, act_from=None, ta
     _lib.check(_lib.lib().e2h_gemm_f32(C.byref(p), _lib.stream()), "e2h_gemm_f32")
 
 
-def linear_packed(x, w, out, *, bias=None, act_from=None, tail=None) -> int:
+def linear_packed(x, w, out, *, bias=None, act_from=None, tail=None, act: str = "relu2") -> int:
     """Several projections of x at once: ``out`` [T, F0] takes the first F0 features of ``w`` in
-    x's type (squared ReLU from feature ``act_from`` on), ``tail`` [T, F - F0] the others in fp32;
-    ``bias`` fp32 [F]. Returns the number of launches."""
+    x's type (activation ``act`` from feature ``act_from`` on), ``tail`` [T, F - F0] the others in
+    fp32; ``bias`` fp32 [F]. Returns the number of launches."""
     F0, F = out.shape[1], w.shape[0]
     if x.dtype == torch.float32:
         _gemm_f32(w, x, epi=EPI_STORE_F32, out=out, bias=bias, act_from=act_from, tail=tail,
-                  tail_from=F0 if F > F0 else 0)
+                  tail_from=F0 if F > F0 else 0, act=act)
         return 1
     if F > F0 and x.shape[0] <= 128:
         gemm(w, x, epi=EPI_STORE_BF16, out=out, bias=bias, act_from=act_from, tail=tail,
-             tail_from=F0)
+             tail_from=F0, act=act)
         return 1
-    gemm(w[:F0], x, epi=EPI_STORE_BF16, out=out, bias=bias, act_from=act_from)
+    gemm(w[:F0], x, epi=EPI_STORE_BF16, out=out, bias=bias, act_from=act_from, act=act)
     if F == F0:
         return 1
     # many tokens: the few tail features would break the large tiles of the main product
@@ -499,12 +529,26 @@ def linear_residual_f32(x, w, residual) -> None:
         gemm(w, x, epi=EPI_RESIDUAL_F32, out=residual, aux=residual)
 
 
-def linear_f32_out(x, w, out) -> None:
-    """out (fp32) = x @ w^T."""
+def linear_f32_out(x, w, out, scale: float = 1.0, softcap: float = 0.0, bias=None) -> None:
+    """out (fp32) = (x @ w^T + bias) * scale, then softcap * tanh(out / softcap) unless ``softcap`` is
+    0."""
+    kw = dict(epi=EPI_STORE_F32, out=out, out_scale=scale, softcap=softcap, bias=bias)
+    _gemm_f32(w, x, **kw) if x.dtype == torch.float32 else gemm(w, x, **kw)
+
+
+def batched_linear(x, w, out, *, batch: int, k: int, x_step: int, out_step: int,
+                   gate: bool = False) -> None:
+    """One product per head: ``w`` holds ``batch`` matrices [F, k] below one another; matrix g takes
+    the columns g * x_step .. + k of x [T, *] to the columns g * out_step .. + F of out [T, *].
+    ``gate``: out holds gate inputs and receives product * sigmoid(gate). In bf16 the steps are
+    multiples of 8 and x is finite in all its columns."""
+    assert w.shape[1] == k and x.shape[1] >= (batch - 1) * x_step + k
+    assert w.shape[0] % batch == 0 and out.shape[1] >= (batch - 1) * out_step + w.shape[0] // batch
+    kw = dict(out=out, batch=(batch, x_step, out_step))
     if x.dtype == torch.float32:
-        _gemm_f32(w, x, epi=EPI_STORE_F32, out=out)
+        _gemm_f32(w, x[:, :k], epi=EPI_GATE if gate else EPI_STORE_F32, **kw)
     else:
-        gemm(w, x, epi=EPI_STORE_F32, out=out)
+        gemm(w, x[:, :k], epi=EPI_GATE if gate else EPI_STORE_BF16, **kw)
 
 
 def grouped_swiglu(x, w1, w3, out, group_off, n_groups: int, group_tmax: int) -> None:
@@ -514,9 +558,12 @@ def grouped_swiglu(x, w1, w3, out, group_off, n_groups: int, group_tmax: int) ->
     _gemm_f32(w1, x, **kw) if x.dtype == torch.float32 else gemm(w1, x, **kw)
 
 
-def grouped_linear(x, w, out, group_off, n_groups: int, group_tmax: int) -> None:
-    """Rows of group g: x @ w[g]^T."""
+def grouped_linear(x, w, out, group_off, n_groups: int, group_tmax: int,
+                   act: Optional[str] = None) -> None:
+    """Rows of group g: x @ w[g]^T, through the activation ``act`` if one is named."""
     kw = dict(out=out, group_off=group_off, n_groups=n_groups, group_tmax=group_tmax)
+    if act:
+        kw.update(act=act, act_from=0)
     if x.dtype == torch.float32:
         _gemm_f32(w, x, epi=EPI_STORE_F32, **kw)
     else:
