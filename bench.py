@@ -16,7 +16,8 @@ with CUDA events between barriers, max over ranks.
 prompt copied from pinned host memory and the generated tokens copied back to pinned host memory
 inside the timed region of every step.
 
-``--workload bovinex`` measures the hybrid decoder beside the LLaMA path at equal size instead.
+``--workload bovinex`` measures that hybrid decoder beside the LLaMA path at equal size instead,
+``--workload ruralorn`` that one beside the Bovinex attention + expert layers at equal size.
 
 ``--impl reference`` runs the unmodified reference from ``baseline/_ref`` (its ``Transformer``,
 ``apply_tp`` and ``generate`` with its ``torch.compile``'d decode step) on the same workload.
@@ -58,11 +59,13 @@ def parse():
     ap.add_argument("--warmup", type=int, default=3)
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
     ap.add_argument("--workload", default="decode", choices=["decode", "sft", "prm",
-                                                                       "bovinex"],
+                                                                       "bovinex", "ruralorn"],
                     help="decode: batched generation (headline); sft: full-parameter SFT step; "
                     "bovinex: prefill and decode throughput of the hybrid decoder beside the LLaMA "
-                    "path at equal size")
-    ap.add_argument("--size", default="4k", choices=["2k", "4k"], help="bovinex: layer shapes")
+                    "path at equal size; ruralorn: the same beside the Bovinex attention + expert "
+                    "layers at equal size")
+    ap.add_argument("--size", default="4k", choices=["2k", "4k"],
+                    help="bovinex, ruralorn: layer shapes")
     ap.add_argument("--quant", default="none", choices=["none", "int8", "int4"],
                     help="decode: weight-only quantisation of the linears (int4: groups of 128)")
     ap.add_argument("--micro", type=int, default=16, help="sft: sequences per micro batch")
@@ -606,16 +609,27 @@ def run_ours_prm(a):
 HYBRID_BATCH, HYBRID_PROMPT, HYBRID_DECODE, HYBRID_LAYERS = 64, 1024, 64, 8
 
 
-def run_bovinex(a):
-    """Prefill and decode throughput of the Bovinex hybrid decoder (8 layers of the named size,
-    random weights) and of the LLaMA path at equal size (same width, heads, layers and active
-    feed-forward parameters), both through their engines: a step is one batch of 64 prompts of
-    1024 tokens, then 64 captured decode steps. ``value`` = Bovinex decode tokens/s; the e2e number
-    is the same generation through inference_generate.generate with host inputs and outputs."""
+# workload -> (model of bench/hybrid_shapes.py beside it, key of its numbers, what the model is)
+HYBRID_RUNS = {
+    "bovinex": ("llama", "llama_equal_size",
+                "attention / gated linear attention, dense / 8 experts top 2"),
+    "ruralorn": ("bovinex_attention", "bovinex_equal_size",
+                 "latent attention, 8 experts top 2 beside a shared one"),
+}
+
+
+def run_hybrid(a):
+    """Prefill and decode throughput of a hybrid decoder (8 layers of the named size, random weights)
+    and of the framework's closest other model at equal size (Bovinex: the LLaMA path; Ruralorn:
+    Bovinex attention + expert layers), both through their engines: a step is one batch of 64
+    prompts of 1024 tokens, then 64 captured decode steps. ``value`` = the design's decode tokens/s;
+    the e2e number is the same generation through inference_generate.generate with host inputs and
+    outputs."""
     import torch
     rank, local, world = dist_setup(a.gpus)
     if world > 1:
-        raise SystemExit("the bovinex workload runs on one GPU")
+        raise SystemExit("the hybrid decoders' workloads run on one GPU")
+    other, other_key, about = HYBRID_RUNS[a.workload]
     sys.path.insert(0, os.path.join(ROOT, "bench"))
     import hybrid_shapes
     import inference_generate as api
@@ -628,7 +642,7 @@ def run_bovinex(a):
     host_out = torch.empty(B, P + N + 1, dtype=torch.int32).pin_memory()
     sampler, res, launches = ClockSampler(local), {}, 0
     sampler.start()
-    for name in ("bovinex", "llama"):
+    for name in (a.workload, other):
         build = getattr(hybrid_shapes, f"{name}_model")
         model = build(a.size, HYBRID_LAYERS)
         eng = get_engine(model, B, P + N + 8)
@@ -657,7 +671,7 @@ def run_bovinex(a):
                      "prefill_ms": pre / a.steps, "decode_step_us": dec / a.steps / N * 1e3,
                      "launches_per_decode_step": per_step,
                      "weight_bytes": eng.weight_bytes()}
-        if name == "bovinex":
+        if name == a.workload:
             launches = (eng.prefill_launches + N * per_step) * a.steps
 
             def e2e(i):
@@ -673,19 +687,19 @@ def run_bovinex(a):
         del model, eng, g
         torch.cuda.empty_cache()
     clocks = sampler.stop()
-    b = res["bovinex"]
+    b = res[a.workload]
     print(json.dumps({
-        "metric": "bovinex_decode_tokens_per_s", "value": b["decode_tokens_per_s"],
+        "metric": f"{a.workload}_decode_tokens_per_s", "value": b["decode_tokens_per_s"],
         "unit": "tokens/s", "n_gpus": 1, "steps": a.steps, "warmup": a.warmup,
         "ms_per_step": b["prefill_ms"] + b["decode_step_us"] * N / 1e3, "higher_is_better": True,
         "scaling": "strong", "vs_baseline": None, "dtype": "bf16",
         "data": "synthetic (random token ids, random-init weights)", "impl": "ours",
-        "config": {"model": f"Bovinex {a.size}: {HYBRID_LAYERS} layers, attention / gated linear "
-                            "attention, dense / 8 experts top 2 (bench/hybrid_shapes.py)",
+        "config": {"model": f"{a.workload.capitalize()} {a.size}: {HYBRID_LAYERS} layers, {about} "
+                            "(bench/hybrid_shapes.py)",
                    "global_batch": B, "seq_len": P + N, "prompt_len": P, "decode_steps": N,
                    "parallelism": "tp1",
                    "l2": "inputs larger than L2 (weights and caches stream per step)"},
-        "bovinex": b, "llama_equal_size": res["llama"], "clocks": clocks,
+        a.workload: b, other_key: res[other], "clocks": clocks,
         "e2e": {"value": B * (N + 1) * a.steps / (ms_e2e / 1e3), "unit": "tokens/s",
                 "h2d_bytes_per_step": B * P * 4, "d2h_bytes_per_step": B * (P + N + 1) * 4},
         "gpu_launches": launches, "kernel_status": _lib.read_status()}), flush=True)
@@ -708,7 +722,7 @@ def run_reference(a):
         from baseline import reference_runner, reference_sft_runner
     except Exception as e:  # noqa: BLE001
         return unavailable(f"reference runner import failed: {type(e).__name__}: {e}")
-    if a.workload == "bovinex":
+    if a.workload in HYBRID_RUNS:
         return unavailable("the reference has no such model")
     if a.workload == "prm":
         return unavailable("no reference arm is wired for the reward-model training workload")
@@ -733,8 +747,8 @@ if __name__ == "__main__":
         run_ours_sft(args)
     elif args.workload == "prm":
         run_ours_prm(args)
-    elif args.workload == "bovinex":
-        run_bovinex(args)
+    elif args.workload in HYBRID_RUNS:
+        run_hybrid(args)
     else:
         run_ours(args)
     finish()

@@ -1,7 +1,10 @@
 """Device time of every kernel of a hybrid-decoder layer against its roofline, beside the like
 kernels of the LLaMA path at equal size.
 
-    python bench/hybrid_kernel_bench.py [--size 4k] [--batch 64] [--context 1024] [--prompt 8x2048]
+    python bench/hybrid_kernel_bench.py [--model bovinex|ruralorn] [--size 4k] [--batch 64]
+                                        [--context 1024] [--prompt 8x2048]
+
+Beside Bovinex: the LLaMA path; beside Ruralorn: the Bovinex layers of attention + experts.
 
 Each kernel is timed alone with CUDA events, L2 flushed before every launch (a 512 MB write),
 median of the launches. The roofline time is the larger of algorithmic bytes over the measured copy
@@ -20,7 +23,8 @@ sys.path.insert(0, os.path.join(ROOT, "bench"))
 
 import torch  # noqa: E402
 
-from hybrid_shapes import bovinex_model, llama_model  # noqa: E402
+from hybrid_shapes import (bovinex_attention_model, bovinex_model, llama_model,  # noqa: E402
+                           ruralorn_model)
 
 
 def peaks():
@@ -70,10 +74,11 @@ def i32(x):
     return torch.tensor(x, dtype=torch.int32, device="cuda")
 
 
-def bovinex(size, batch, context, prompts, plen):
+def bovinex(size, batch, context, prompts, plen, attention_only=False):
     from easy_to_hard_b200.models.hybrid_engine import _Scratch
     from easy_to_hard_b200.ops import gemm, hybrid as hy
-    model = bovinex_model(size, 4)
+    layers = 1 if attention_only else 4
+    model = bovinex_attention_model(size, 1) if attention_only else bovinex_model(size, 4)
     n_max = prompts * plen
     eng = model.make_engine(max(batch, prompts), max(context + 8, plen), use_graph=False)
     cfg, W = model.config, model.config.dim
@@ -93,7 +98,7 @@ def bovinex(size, batch, context, prompts, plen):
         hy.stream_norm(w.x, model.layers[0].norm1, h, eps=1e-5, offset=1.0)
         row("residual norm", time_us(lambda: hy.stream_norm(
             w.x, model.layers[0].norm1, h, eps=1e-5, offset=1.0)), n * W * 6)
-        for li in range(4):
+        for li in range(layers):
             blk, mix, m, f = (model.layers[li], eng.mixers[li], model.layers[li].layer.mixer,
                               model.layers[li].layer.mlp)
             tag = f"{m.kind}+{f.kind}"
@@ -140,7 +145,7 @@ def bovinex(size, batch, context, prompts, plen):
                 time_us(lambda: gemm.linear_residual_f32(act[:, blk.off_g:], blk.mat("w_out"),
                                                          w.x[:n])),
                 (W * K + n * K) * 2 + n * W * 8, 2.0 * n * W * K)
-            if f.kind == "moe" and li == 1:
+            if f.kind == "moe" and li == layers // 3:
                 top, E = f.top, f.experts
                 place, ew = w.choice(n, top)
                 hg, ag, y = w.hg[: n * top, :W], w.ag(n * top, blk.ffp), w.y[: n * top, :W]
@@ -162,6 +167,100 @@ def bovinex(size, batch, context, prompts, plen):
                 row("residual norm + expert outputs", time_us(lambda: hy.stream_norm(
                     w.x, model.layers[0].norm1, h, eps=1e-5, offset=1.0,
                     experts=(y, place, ew))), n * W * (10 + 2 * top))
+        del w
+    from easy_to_hard_b200.ops import _lib
+    assert _lib.read_status() == 0
+
+
+def ruralorn(size, batch, context, prompts, plen):
+    from easy_to_hard_b200.models.hybrid_engine import _Scratch
+    from easy_to_hard_b200.ops import gemm, hybrid as hy
+    model = ruralorn_model(size, 1)
+    eng = model.make_engine(max(batch, prompts), max(context + 8, plen), use_graph=False)
+    W, blk, mix = model.config.dim, model.layers[0], eng.mixers[0]
+    m, f = blk.layer.mixer, blk.layer.mlp
+    H, d, r, e, k = m.heads, m.dim, m.rot_dim, m.vdim, m.kv_rank
+    for phase, n in (("decode", batch), ("prompt", prompts * plen)):
+        head(f"Ruralorn {size}, {phase}: " + (f"{batch} sequences at position {context}"
+                                              if phase == "decode" else
+                                              f"{prompts} prompts of {plen} tokens"))
+        w = _Scratch(model, n)
+        w.x.normal_()
+        h = w.h[:n, :W]
+        norm = lambda **kw: hy.stream_norm(w.x, blk.norm1, w.h[:n], eps=1e-5, **kw)  # noqa: E731
+        norm()
+        row("residual norm", time_us(norm), n * W * 6)
+        act, F = w.act(n, blk.f_main), blk.f_main
+        run = lambda: gemm.linear_packed(h, blk.mat("w_in"), act)  # noqa: E731
+        run()
+        row(f"w_in GEMM: q, latent, gate ({F} x {W})", time_us(run), (F * W + n * W + n * F) * 2,
+            2.0 * n * F * W)
+        if phase == "decode":
+            pos, slot = i32([context] * n), i32(list(range(n)))
+            ql, ol = eng._absorbed_rows(mix, n)
+            run = lambda: mix.absorb(act, ql)  # noqa: E731
+            run()
+            row(f"absorbed queries ({H} x {k} x {d})", time_us(run),
+                (H * k * d + n * H * (d + k)) * 2, 2.0 * n * H * k * d)
+            keys = min(context + 1, m.window or context + 1)
+            row("attention decode (norm, rotation, cache write)", time_us(
+                lambda: mix.attend(act, ql, ol, pos, slot, fused=True)),
+                n * (keys * (k + r) + H * (2 * k + r) + k + r) * 2, 2.0 * n * keys * H * (2 * k + r))
+            row(f"value expansion + gate ({H} x {e} x {k})", time_us(lambda: mix.values(act, ol)),
+                (H * k * e + n * H * (k + 2 * e)) * 2, 2.0 * n * H * k * e)
+        else:
+            pos = i32(list(range(plen)) * prompts)
+            slot = i32([b for b in range(prompts) for _ in range(plen)])
+            seg = i32([b * plen for b in range(prompts + 1)])
+            ctx = eng._context([plen] * prompts, [0] * prompts, list(range(prompts)))
+            bf = dict(dtype=torch.bfloat16, device="cuda")
+            rows, kv = torch.empty(n, k + r, **bf), torch.empty(n, blk.w_kv.shape[0], **bf)
+            row("attention prep (norm, rotation, cache write)", time_us(
+                lambda: mix.prep(act, pos, slot, ctx, rows)), n * (3 * (k + r) + 2 * H * r) * 2)
+            row(f"key and value expansion ({H * (d + e)} x {k})", time_us(
+                lambda: mix.expand(rows, kv)), (H * (d + e) * k + n * (H * (d + e) + k)) * 2,
+                2.0 * n * H * (d + e) * k)
+            vis = sum(min(i + 1, m.window or plen) for i in range(plen)) * prompts
+            row("attention (windowed flash, gate)", time_us(
+                lambda: mix.flash(act, pos, slot, seg, ctx, rows, kv)),
+                n * (H * (d + r + 2 * e) + H * (d + e) + r) * 2, 2.0 * vis * H * (d + r + e))
+        K = blk.f_main - blk.off_g
+        row(f"w_out GEMM + fp32 residual ({W} x {K})", time_us(
+            lambda: gemm.linear_residual_f32(act[:, blk.off_g:], blk.mat("w_out"), w.x[:n])),
+            (W * K + n * K) * 2 + n * W * 8, 2.0 * n * W * K)
+        up, tail, top, E = w.ff(n, blk.f_ff), w.tail(n, blk.n_ff_tail), f.top, f.experts
+        F = blk.w_ff.shape[0]
+        run = lambda: gemm.linear_packed(h, blk.mat("w_ff"), up, tail=tail, act="gelu",  # noqa: E731
+                                         act_from=0)
+        run()
+        row(f"w_ff GEMM: shared up + GELU, router ({F} x {W})", time_us(run),
+            (F * W + n * W + n * F) * 2, 2.0 * n * F * W)
+        row(f"w_down GEMM + fp32 residual ({W} x {blk.f_ff})", time_us(
+            lambda: gemm.linear_residual_f32(up, blk.mat("w_down"), w.x[:n])),
+            (W * blk.f_ff + n * blk.f_ff) * 2 + n * W * 8, 2.0 * n * W * blk.f_ff)
+        place, ew = w.choice(n, top)
+        hg, ag, y = w.hg[: n * top, :W], w.ag(n * top, blk.ffp), w.y[: n * top, :W]
+        tail.normal_()
+        run = lambda: hy.moe_route(tail[:, blk.off_r:], E, top, h, hg, w.off, place, ew,  # noqa: E731
+                                   w.sel, score=f.score, weight_input=True)
+        row("expert routing + weighted regrouping", time_us(run), n * W * 2 * (1 + top))
+        run()
+        live = min(E, n * top)
+        row(f"expert up + GELU ({E} x {blk.ffp} x {W})", time_us(
+            lambda: gemm.grouped_linear(hg, blk.mat("e_up"), ag, w.off, E, n, act="gelu")),
+            (live * blk.ffp * W + n * top * (W + blk.ffp)) * 2, 2.0 * n * top * blk.ffp * W)
+        row(f"expert down ({E} x {W} x {blk.ffp})", time_us(
+            lambda: gemm.grouped_linear(ag, blk.mat("e_down"), y, w.off, E, n)),
+            (live * blk.ffp * W + n * top * (W + blk.ffp)) * 2, 2.0 * n * top * blk.ffp * W)
+        row("residual norm + expert outputs", time_us(lambda: norm(experts=(y, place, None))),
+            n * W * (10 + 2 * top))
+        V = model.head_w.shape[0]
+        nl = min(n, batch)
+        logits = torch.empty(nl, V, device="cuda")
+        row(f"LM head + scale, soft cap ({V} x {W}, {nl} rows)", time_us(
+            lambda: gemm.linear_f32_out(h[:nl], model.head_w[:, :W], logits, scale=0.5,
+                                        softcap=30.0)),
+            (V * W + nl * W) * 2 + nl * V * 4, 2.0 * nl * V * W)
         del w
     from easy_to_hard_b200.ops import _lib
     assert _lib.read_status() == 0
@@ -214,6 +313,7 @@ def llama(size, batch, context, prompts, plen):
 
 if __name__ == "__main__":
     ap = argparse.ArgumentParser()
+    ap.add_argument("--model", default="bovinex", choices=["bovinex", "ruralorn"])
     ap.add_argument("--size", default="4k")
     ap.add_argument("--batch", type=int, default=64)
     ap.add_argument("--context", type=int, default=1024)
@@ -221,6 +321,11 @@ if __name__ == "__main__":
     a = ap.parse_args()
     p, t = (int(v) for v in a.prompt.split("x"))
     with torch.no_grad():
-        bovinex(a.size, a.batch, a.context, p, t)
-        torch.cuda.empty_cache()
-        llama(a.size, a.batch, a.context, p, t)
+        if a.model == "ruralorn":
+            ruralorn(a.size, a.batch, a.context, p, t)
+            torch.cuda.empty_cache()
+            bovinex(a.size, a.batch, a.context, p, t, attention_only=True)
+        else:
+            bovinex(a.size, a.batch, a.context, p, t)
+            torch.cuda.empty_cache()
+            llama(a.size, a.batch, a.context, p, t)

@@ -1,5 +1,7 @@
-"""Layer shapes of the hybrid-decoder benchmarks: Bovinex configurations whose layers resemble a
-real model's, and LLaMA configurations of equal size (same width, query heads, kv heads, layers and
+"""Layer shapes of the hybrid-decoder benchmarks: Bovinex and Ruralorn configurations whose layers
+resemble a real model's, LLaMA configurations of the size of the Bovinex ones (same width, query
+heads, kv heads, layers and active feed-forward parameters), and Bovinex configurations of the size of
+the Ruralorn ones (attention and expert layers only; same width, query heads, window, experts and
 active feed-forward parameters)."""
 from __future__ import annotations
 
@@ -15,8 +17,9 @@ SIZES = {
 }
 
 
-def bovinex_config(size: str, layers: int = 8):
-    """attention + dense, gla + experts, gla + dense, attention + experts, repeated."""
+def bovinex_config(size: str, layers: int = 8, attention_only: bool = False):
+    """attention + dense, gla + experts, gla + dense, attention + experts, repeated; or attention +
+    experts only."""
     from easy_to_hard_b200.models.hybrid import (AttentionMixer, DenseMlp, GlaMixer, HybridConfig,
                                                  HybridLayer, MoeMlp, Rotary, Yarn)
     W, H, G, win, gh, ff, E, top, eff, _, vocab = SIZES[size]
@@ -29,6 +32,8 @@ def bovinex_config(size: str, layers: int = 8):
         return GlaMixer(gh, 128, 256, 16.0, 16)
     kinds = [(att, DenseMlp(ff)), (gla, MoeMlp(E, top, eff)), (gla, DenseMlp(ff)),
              (att, MoeMlp(E, top, eff))]
+    if attention_only:
+        kinds = kinds[3:] * 4
     return HybridConfig("Bovinex", vocab, W, 1e-5, W ** 0.5,
                         [HybridLayer(kinds[i % 4][0](), kinds[i % 4][1]) for i in range(layers)],
                         norm_offset=1.0)
@@ -37,6 +42,38 @@ def bovinex_config(size: str, layers: int = 8):
 def bovinex_model(size: str, layers: int = 8):
     from easy_to_hard_b200.models.hybrid import HybridLM
     return HybridLM.random(bovinex_config(size, layers))
+
+
+def bovinex_attention_model(size: str, layers: int = 8):
+    from easy_to_hard_b200.models.hybrid import HybridLM
+    return HybridLM.random(bovinex_config(size, layers, attention_only=True))
+
+
+# latent rank, dim, rotated dim, value dim of a head; expert ff and shared ff (two matrices each) with
+# as many active parameters as the gated experts of the Bovinex shapes
+LATENT = (512, 128, 64, 128)
+RURALORN_FF = {"2k": (3440, 1376), "4k": (6880, 2752)}
+
+
+def ruralorn_config(size: str, layers: int = 8):
+    from easy_to_hard_b200.models.hybrid import (DenseMlp, HybridConfig, HybridLayer, LatentMixer,
+                                                 MoeMlp, Rotary)
+    W, H, _, win, _, _, E, top, _, _, vocab = SIZES[size]
+    rank, dim, rot, vdim = LATENT
+    ff, shared = RURALORN_FF[size]
+
+    def layer():
+        return HybridLayer(LatentMixer(H, dim, rot, vdim, rank, (dim + rot) ** -0.5,
+                                       Rotary(rot, 1e6, interleaved=True), win),
+                           MoeMlp(E, top, ff, gated=False, act="gelu", score="sigmoid",
+                                  weight_input=True, bias=False, shared=DenseMlp(shared, "gelu")))
+    return HybridConfig("Ruralorn", vocab, W, 1e-5, W ** 0.5, [layer() for _ in range(layers)],
+                        parallel=False, logit_scale=0.5, logit_softcap=30.0)
+
+
+def ruralorn_model(size: str, layers: int = 8):
+    from easy_to_hard_b200.models.hybrid import HybridLM
+    return HybridLM.random(ruralorn_config(size, layers))
 
 
 def llama_model(size: str, layers: int = 8):
