@@ -19,10 +19,10 @@
 //                 earlier positions there from the cache; rotates q in place. One CTA per row.
 //   latent_attn   absorbed attention, one token per cluster of CTAs: its keys are split over the CTAs
 //                 and merged through distributed shared memory.
-//     bf16        warp-level matrix products on a ring of cache rows that bulk copies fill. A token
-//                 brings at most 16 or 32 query rows, far below a tcgen05 tile, and the kernel is a
-//                 stream of the cache; in its fused form (decode) it also does the work of
-//                 latent_prep. Prompts expand the keys and use flash_window.cu instead.
+//     bf16        warp-level matrix products on a ring of cache rows that TMA fills. A token brings
+//                 at most 16 or 32 query rows, far below a tcgen05 tile, and the kernel is a stream of
+//                 the cache; in its fused form (decode) it also does the work of latent_prep.
+//                 Prompts expand the keys and use flash_window.cu instead.
 //     any         fp32, and sizes the other form does not take: one warp per head on CUDA cores.
 #include <cooperative_groups.h>
 #include <cuda_bf16.h>
@@ -32,6 +32,7 @@
 #include <string.h>
 #include <mutex>
 
+#include "flash_common.cuh"
 #include "launch.cuh"
 #include "ptx.cuh"
 #include "scalar_types.cuh"
@@ -248,7 +249,11 @@ __global__ void __launch_bounds__(kLatHeads * 32) latent_attn_kernel(const Laten
 }
 
 // ------------------------------------------------------------------ bf16 form
-constexpr int kMmaThreads = 256, kMmaKeys = 64, kPartPitch = 72, kProbPitch = 72;
+constexpr int kMmaThreads = 256;
+constexpr int kMmaKeys = 64, kMmaRows = 32, kMmaStages = 5;    // keys of a tile; rows of a stage, stages
+constexpr int kMmaSmem = 224 * 1024;             // dynamic shared memory; some 2 KB are static
+constexpr int kPartPitch = 72, kProbPitch = 72;
+constexpr int kMmaBlock = kMmaRows * 128;        // 64 columns of a stage's rows, 128-byte swizzle
 
 __device__ __forceinline__ void ldsm4(uint32_t* r, uint32_t addr) {
   asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"
@@ -265,171 +270,200 @@ __device__ __forceinline__ void mma16816(float* c, const uint32_t* a, uint32_t b
       : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
       : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
 }
-// stream: the row is read once per step (L2 evict-first)
-__device__ __forceinline__ void bulk_row(uint32_t dst, const void* src, uint32_t bytes, uint32_t bar,
-                                         bool stream, uint64_t policy) {
-  if (stream)
-    asm volatile(
-        "cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes.L2::cache_hint "
-        "[%0], [%1], %2, [%3], %4;"
-        ::"r"(dst), "l"(src), "r"(bytes), "r"(bar), "l"(policy)
-        : "memory");
-  else
-    asm volatile(
-        "cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];"
-        ::"r"(dst), "l"(src), "r"(bytes), "r"(bar)
-        : "memory");
+__device__ __forceinline__ void cp_async16(uint32_t dst, const void* src) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst), "l"(src) : "memory");
+}
+__device__ __forceinline__ void cp_async_wait_all() {
+  asm volatile("cp.async.wait_all;" ::: "memory");
 }
 
-// Shared memory of a CTA with R = 16 MT query rows.
+// Shared memory of a CTA with R = 16 MT query rows: the ring of key rows, the parts of the scores, the
+// probabilities, the token's own row. The query rows start where the parts and probabilities are
+// later; the output tile takes the place of the ring.
 struct LatentPlan {
-  int kd16, pitch;           // row length rounded up to a k-step; row distance (elements), 16 bytes
-                             // past a multiple of 32 so that ldmatrix rows fall on all banks
-  int stage, part, prob, nk, total;   // byte offsets
+  int kd16, pitch;           // row length rounded up to a k-step; distance of query rows (elements), 16
+                             // bytes past a multiple of 32 so that ldmatrix rows fall on all banks
+  int stage, part, prob, own, total;   // bytes of a stage; byte offsets
   __host__ __device__ LatentPlan(int kd, int rank, int mt) {
     const int R = 16 * mt;
     kd16 = (kd + 15) / 16 * 16;
     pitch = kd16 + 8;
-    stage = 0;
-    int end = 2 * kMmaKeys * pitch * 2;
-    const int out = R * (rank + 4) * 4;           // the output tile takes the place of the ring
-    if (end < out) end = out;
-    part = (end + 15) / 16 * 16;                  // score parts; the query rows before them
+    stage = (kd + 63) / 64 * kMmaBlock;
+    part = kMmaStages * stage;
+    const int out = R * (rank + 4) * 4;
+    if (part < out) part = (out + 1023) / 1024 * 1024;
     prob = part + 4 * R * kPartPitch * 4;
-    nk = prob + R * kProbPitch * 2;
+    own = prob + R * kProbPitch * 2;
     const int q = part + R * pitch * 2;
-    if (nk < q) nk = q;
-    total = nk + pitch * 2;
+    if (own < q) own = q;
+    total = own + kd16 * 2;
   }
 };
+
+// Column c of row r of a stage.
+__device__ __forceinline__ uint32_t tile_at(uint32_t tile, int r, int c) {
+  return tile + (c >> 6) * kMmaBlock + r * 128 + ((((c >> 3) ^ r) & 7) << 4) + (c & 7) * 2;
+}
 
 // MT: blocks of 16 query heads; KQ: 16-column steps of a row per warp (a quarter of the row); NP: pairs
 // of 8-column tiles of the latent per warp.
 //
-// Work of the eight warps on a tile of 64 keys: scores - warp (quarter of the columns, half of the
-// keys), its query fragments stay in registers; the four partial scores of a (head, key) meet in
-// shared memory, where 256 / R threads run the softmax of a head; output - warp (1/8 of the latent
-// columns, all keys). Every byte of a cache row is read twice from shared memory, once per product.
+// TMA fills the ring 32 rows at a time (rows past the last key are read and masked), a stage as soon as
+// every warp is past the tile that read it last. Work of the eight warps on a tile of 64 keys: scores - warp (quarter of the columns,
+// half of the keys), its query fragments stay in registers; the four partial scores of a (head, key)
+// meet in shared memory, where 256 / R threads run the softmax of a head; output - warp (1/8 of the
+// latent columns, all keys). Every byte of a cache row is read twice from shared memory, once per
+// product. Two barriers per tile.
 template <int MT, int KQ, int NP, bool FUSED>
-__global__ void __launch_bounds__(kMmaThreads, 1) latent_attn_mma_kernel(const LatentParams p) {
+__global__ void __launch_bounds__(kMmaThreads, 1)
+latent_attn_mma_kernel(const __grid_constant__ CUtensorMap tm, const int boxes,
+                       const LatentParams p) {
   using T = __nv_bfloat16;
   constexpr int R = 16 * MT, TPR = kMmaThreads / R, KPT = kMmaKeys / TPR;
-  extern __shared__ __align__(128) uint8_t lat_b[];
-  __shared__ __align__(8) uint64_t full[2];
+  static_assert(KPT % 4 == 0, "keys of a softmax thread come in fours");
+  extern __shared__ __align__(1024) uint8_t lat_raw[];
+  uint8_t* lat_b = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(lat_raw) + 1023) &
+                                              ~uintptr_t(1023));
+  __shared__ __align__(8) uint64_t full[kMmaStages];
   __shared__ float red[33];
   __shared__ float alpha_s[R], fin[R][2];
   __shared__ int abort_s;
   const int kd = p.rank + p.rot;
   const LatentPlan plan(kd, p.rank, MT);
   const int pitch = plan.pitch;
-  T* ring = reinterpret_cast<T*>(lat_b + plan.stage);
   float* part_s = reinterpret_cast<float*>(lat_b + plan.part);
   T* q_s = reinterpret_cast<T*>(lat_b + plan.part);
   T* prob_s = reinterpret_cast<T*>(lat_b + plan.prob);
-  T* new_s = reinterpret_cast<T*>(lat_b + plan.nk);
+  T* own_s = reinterpret_cast<T*>(lat_b + plan.own);
 
   cg::cluster_group cluster = cg::this_cluster();
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   if (tid == 0) {
-    mbar_init(smem_u32(&full[0]), 1);
-    mbar_init(smem_u32(&full[1]), 1);
+    for (int s = 0; s < kMmaStages; ++s) mbar_init(smem_u32(&full[s]), 1);
     abort_s = 0;
     fence_mbar_init();
+    tma_prefetch_desc(&tm);
   }
-  // columns past a row's end are multiplied by zero: they have to be numbers
-  for (int i = tid; i < 2 * kMmaKeys; i += kMmaThreads)
-    for (int d = kd; d < pitch; d += 8)
-      *reinterpret_cast<uint4*>(ring + i * pitch + d) = make_uint4(0, 0, 0, 0);
   __syncthreads();
   pdl_launch_dependents();
   pdl_wait_prior();
 
   const int rank = blockIdx.x, h0 = blockIdx.y * R, t = blockIdx.z;
   const int nr = min(R, p.H - h0);
+  const bool has_own = FUSED && rank == p.splits - 1;   // holds the token's own key
+  const T* act = static_cast<const T*>(p.act) + t * p.ld;
+  // every load that does not depend on the position first: indices, query rows, own latent, norm
   int pos = p.pos[t], slot = p.slot[t];
+  const int qv = p.rank / 8;
+  for (int i = tid; i < nr * qv; i += kMmaThreads) {
+    const int r = i / qv, d = (i - r * qv) * 8;
+    cp_async16(smem_u32(q_s + r * pitch + d),
+               static_cast<const T*>(p.ql) + ((long long)t * p.H + h0 + r) * p.rank + d);
+  }
+  const int per = (plan.kd16 - p.rank) / 8;      // pieces of a query row behind the latent columns
+  auto piece = [&](int i, int& r, int& d) -> const T* {
+    r = i / max(per, 1);
+    d = (i - r * per) * 8;
+    return i < R * per && r < nr && d < p.rot
+               ? act + p.off_q + (h0 + r) * (p.dim + p.rot) + p.dim + d : nullptr;
+  };
+  int r0, d0;
+  const T* src0 = piece(tid, r0, d0);
+  const uint4 zero4 = make_uint4(0, 0, 0, 0);
+  const uint4 x0 = src0 ? *reinterpret_cast<const uint4*>(src0) : zero4;
+  const int oc = tid * 8;                        // columns of the own row (at most 576)
+  float own[8], wn[8];
+  if (has_own && oc < kd) {
+    load8(act + p.off_c + oc, own);
+    if (oc < p.rank) load8(p.norm + oc, wn);
+  }
+
   const bool ok = pos >= 0 && pos < p.smax && slot >= 0 && slot < p.slots;
   if (!ok) {                                     // indices come from device memory
     if (tid == 0) atomicCAS(p.status, 0, kStatusBadArgs);
     pos = min(max(pos, 0), p.smax - 1);
     slot = min(max(slot, 0), p.slots - 1);
   }
-  T* cache = static_cast<T*>(p.cache) + (long long)slot * p.smax * kd;
-  const T* act = static_cast<const T*>(p.act) + t * p.ld;
-  const float* cs = p.rot_table + (long long)pos * p.rot;
-  const float sl2 = p.scale * 1.4426950408889634f;
-
-  // keys lo .. pos, split over the cluster; the fused form holds the last one itself
+  // keys lo .. pos, split over the cluster
   const int lo = p.window > 0 ? max(pos - p.window + 1, 0) : 0;
   const int n_keys = pos + 1 - lo;
   const int k_begin = lo + (int)((long long)n_keys * rank / p.splits);
   const int k_end = lo + (int)((long long)n_keys * (rank + 1) / p.splits);
+  const int n_loads = (k_end - k_begin + kMmaRows - 1) / kMmaRows;
   const int n_tiles = (k_end - k_begin + kMmaKeys - 1) / kMmaKeys;
-  const bool has_new = FUSED && rank == p.splits - 1;
-  const bool stream = FUSED && gridDim.y == 1;
-  const uint64_t policy = policy_evict_first();
-  auto load_tile = [&](int it) {                 // warp 0
-    const int k0 = k_begin + it * kMmaKeys;
-    const int rows = min(kMmaKeys, k_end - (has_new ? 1 : 0) - k0);
-    const uint32_t bar = smem_u32(&full[it & 1]);
-    if (lane == 0) mbar_expect_tx(bar, max(rows, 0) * kd * 2);
-    __syncwarp();
-    const uint32_t dst = smem_u32(ring + (it & 1) * kMmaKeys * pitch);
-    for (int r = lane; r < rows; r += 32)
-      bulk_row(dst + r * pitch * 2, cache + (long long)(k0 + r) * kd, kd * 2, bar, stream,
-               policy);
+  auto load = [&](int i) {                       // thread 0
+    const int s = i % kMmaStages;
+    const uint32_t bar = smem_u32(&full[s]);
+    mbar_expect_tx(bar, plan.stage);
+    for (int b = 0; b < boxes; ++b)              // one box for all columns if they are whole blocks
+      tma_load_3d(smem_u32(lat_b + s * plan.stage + b * kMmaBlock), &tm, b * 64,
+                  slot * p.smax + k_begin + i * kMmaRows, 0, bar);
   };
-  if (warp == 0) {
-    if (n_tiles > 0) load_tile(0);
-    if (n_tiles > 1) load_tile(1);
-  }
+  if (tid == 0)
+    for (int i = 0; i < min(n_loads, kMmaStages); ++i) load(i);
 
-  // query rows, rotated part included
-  for (int i = tid; i < R * (plan.kd16 / 8); i += kMmaThreads) {
-    const int r = i / (plan.kd16 / 8), d = (i - r * (plan.kd16 / 8)) * 8, h = h0 + r;
-    uint4 x = make_uint4(0, 0, 0, 0);
-    if (r < nr && d < kd) {
-      if (d < p.rank) {
-        x = *reinterpret_cast<const uint4*>(static_cast<const T*>(p.ql) +
-                                            ((long long)t * p.H + h) * p.rank + d);
+  const float* cs = p.rot_table + (long long)pos * p.rot;
+  float f0[8], fo[8];
+  if (FUSED && src0) load8(cs + d0, f0);
+  if (has_own && oc >= p.rank && oc < kd) load8(cs + oc - p.rank, fo);
+  auto put = [&](int r, int d, bool live, uint4 x, const float* f) {
+    if (FUSED && live) {
+      float v[8];
+      load8(reinterpret_cast<const T*>(&x), v);
+      rotate8(v, f);
+      store8(reinterpret_cast<T*>(&x), v);
+    }
+    *reinterpret_cast<uint4*>(q_s + r * pitch + p.rank + d) = x;
+  };
+  if (tid < R * per) put(r0, d0, src0 != nullptr, x0, f0);
+  for (int i = tid + kMmaThreads; i < R * per; i += kMmaThreads) {
+    int r, d;
+    const T* src = piece(i, r, d);
+    float f[8];
+    if (FUSED && src) load8(cs + d, f);
+    put(r, d, src != nullptr, src ? *reinterpret_cast<const uint4*>(src) : zero4, f);
+  }
+  for (int i = nr * qv + tid; i < R * qv; i += kMmaThreads) {
+    const int r = i / qv, d = (i - r * qv) * 8;
+    *reinterpret_cast<uint4*>(q_s + r * pitch + d) = zero4;
+  }
+  if (has_own) {
+    float ss = 0.f;
+    if (oc < p.rank) {
+#pragma unroll
+      for (int e = 0; e < 8; ++e) ss += own[e] * own[e];
+    }
+    const float rstd = 1.f / sqrtf(block_sum(ss, red) / p.rank_n + p.eps);
+    if (oc < kd) {
+      if (oc < p.rank) {
+#pragma unroll
+        for (int e = 0; e < 8; ++e) own[e] *= rstd * wn[e];
       } else {
-        const T* src = act + p.off_q + h * (p.dim + p.rot) + p.dim + (d - p.rank);
-        if constexpr (FUSED) {
-          float v[8], f[8];
-          load8(src, v);
-          load8(cs + d - p.rank, f);
-          rotate8(v, f);
-          store8(reinterpret_cast<T*>(&x), v);
-        } else {
-          x = *reinterpret_cast<const uint4*>(src);
-        }
+        rotate8(own, fo);
       }
-    }
-    *reinterpret_cast<uint4*>(q_s + r * pitch + d) = x;
-  }
-  if (has_new) {
-    const T* c = act + p.off_c;
-    const float rstd = latent_rstd(p, c, red);
-    for (int i = tid * 8; i < plan.kd16; i += kMmaThreads * 8) {
-      float x[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
-      if (i < kd) latent_row8(p, c, i, rstd, cs, x);
-      store8(new_s + i, x);
-      if (ok && blockIdx.y == 0 && i < kd) store8(cache + (long long)pos * kd + i, x);
+      store8(own_s + oc, own);
+      if (ok && blockIdx.y == 0)
+        store8(static_cast<T*>(p.cache) + ((long long)slot * p.smax + pos) * kd + oc, own);
     }
   }
+  cp_async_wait_all();
   __syncthreads();
 
+  const int op = p.rank + 4;                     // row distance of the output tile
+  float* out_s = reinterpret_cast<float*>(lat_b);
   const int ks = plan.kd16 / 16, kq = warp >> 1, kh = warp & 1;   // column quarter, key half
   const int per_q = (ks + 3) / 4;
   const int s_begin = kq * per_q, s_count = max(0, min(per_q, ks - s_begin));
+  const int c8_last = ks * 2 - 2;                // steps past the row repeat its end, times zero
   uint32_t qf[KQ][MT][4];
-  const int lr = lane & 7, lt = lane >> 3;       // row and tile of this lane's ldmatrix address
+  const int lr = lane & 7, lt = lane >> 3;     // row and tile of this lane's ldmatrix address
 #pragma unroll
   for (int s = 0; s < KQ; ++s)
 #pragma unroll
     for (int mt = 0; mt < MT; ++mt) {
       if (s < s_count) {
-        ldsm4(qf[s][mt], smem_u32(q_s + (mt * 16 + (lt & 1) * 8 + lr) * pitch + (s_begin + s) * 16 +
-                                  (lt >> 1) * 8));
+        ldsm4(qf[s][mt], smem_u32(q_s + (mt * 16 + (lt & 1) * 8 + lr) * pitch +
+                                  (s_begin + s) * 16 + (lt >> 1) * 8));
       } else {
 #pragma unroll
         for (int e = 0; e < 4; ++e) qf[s][mt][e] = 0;
@@ -445,26 +479,27 @@ __global__ void __launch_bounds__(kMmaThreads, 1) latent_attn_mma_kernel(const L
 #pragma unroll
         for (int e = 0; e < 4; ++e) acc[a][b][c][e] = 0.f;
   const int g = lane >> 2, c2 = (lane & 3) * 2;
-  const int row = tid / TPR, sub = tid % TPR;    // softmax: head, keys sub, sub + TPR, ...
+  const int row = tid / TPR, sub = tid % TPR;  // softmax: head, keys 4 sub .., 4 (sub + TPR) ..
   const int n_pairs = (p.rank + 15) / 16;
+  const float sl2 = p.scale * 1.4426950408889634f;
   float m = -FLT_MAX, l = 0.f;
-  __syncthreads();                               // the query rows give way to the score parts
+  __syncthreads();                        // the query rows give way to the score parts
 
+  int st[2] = {0, 1};                          // stages of the tile's halves
+  uint32_t ph[2] = {0, 0};
   for (int it = 0; it < n_tiles; ++it) {
-    T* tile = ring + (it & 1) * kMmaKeys * pitch;
-    const int k0 = k_begin + it * kMmaKeys;
-    const int cnt = min(kMmaKeys, k_end - k0);
-    mbar_wait(smem_u32(&full[it & 1]), (it >> 1) & 1, &abort_s, p.status, kStatusTimeoutFull);
-    if (it == n_tiles - 1 && (cnt < kMmaKeys || has_new)) {
-      const int per = plan.kd16 / 8;             // the token's own row, zeros behind the last key
-      for (int i = tid; i < (kMmaKeys - cnt + 1) * per; i += kMmaThreads) {
-        const int r = i / per, d = (i - r * per) * 8;
-        if (r > 0)
-          *reinterpret_cast<uint4*>(tile + (cnt - 1 + r) * pitch + d) = make_uint4(0, 0, 0, 0);
-        else if (has_new)
-          *reinterpret_cast<uint4*>(tile + (cnt - 1) * pitch + d) =
-              *reinterpret_cast<const uint4*>(new_s + d);
-      }
+    const int cnt = min(kMmaKeys, k_end - k_begin - it * kMmaKeys);
+    const bool two = cnt > kMmaRows;           // the second half was loaded
+    const uint32_t half[2] = {smem_u32(lat_b + st[0] * plan.stage),
+                              smem_u32(lat_b + st[1] * plan.stage)};
+    mbar_wait(smem_u32(&full[st[0]]), ph[0], &abort_s, p.status, kStatusTimeoutFull);
+    if (two) mbar_wait(smem_u32(&full[st[1]]), ph[1], &abort_s, p.status, kStatusTimeoutFull);
+    if (has_own && it == n_tiles - 1) {        // the token's own row
+      const uint32_t base = two ? half[1] : half[0];
+      for (int i = tid; i < kd / 8; i += kMmaThreads)
+        *reinterpret_cast<uint4*>(lat_b + (tile_at(base, (cnt - 1) % kMmaRows, i * 8) -
+                                           smem_u32(lat_b))) =
+            *reinterpret_cast<const uint4*>(own_s + i * 8);
       __syncthreads();
     }
     float sc[MT][4][4];
@@ -474,21 +509,22 @@ __global__ void __launch_bounds__(kMmaThreads, 1) latent_attn_mma_kernel(const L
       for (int b = 0; b < 4; ++b)
 #pragma unroll
         for (int e = 0; e < 4; ++e) sc[a][b][e] = 0.f;
+    if (kh == 0 || two) {
+      const uint32_t krow = (kh ? half[1] : half[0]) + ((lt >> 1) * 8 + lr) * 128;
 #pragma unroll
-    for (int s = 0; s < KQ; ++s) {
-      if (s < s_count) {
-        const T* col = tile + (kh * 32 + (lt >> 1) * 8 + lr) * pitch + (s_begin + s) * 16 +
-                       (lt & 1) * 8;
+      for (int s = 0; s < KQ; ++s) {
+        const int c8 = min((s_begin + s) * 2, c8_last) + (lt & 1);   // 8-column group
+        const uint32_t a = krow + (c8 >> 3) * kMmaBlock + (((c8 ^ lr) & 7) << 4);
+        uint32_t b[2][4];
+        ldsm4(b[0], a);
+        ldsm4(b[1], a + 16 * 128);
 #pragma unroll
-        for (int h = 0; h < 2; ++h) {            // 16 keys each
-          uint32_t b[4];
-          ldsm4(b, smem_u32(col + h * 16 * pitch));
+        for (int x = 0; x < 2; ++x)
 #pragma unroll
           for (int mt = 0; mt < MT; ++mt) {
-            mma16816(sc[mt][2 * h], qf[s][mt], b[0], b[1]);
-            mma16816(sc[mt][2 * h + 1], qf[s][mt], b[2], b[3]);
+            mma16816(sc[mt][2 * x], qf[s][mt], b[x][0], b[x][1]);
+            mma16816(sc[mt][2 * x + 1], qf[s][mt], b[x][2], b[x][3]);
           }
-        }
       }
     }
 #pragma unroll
@@ -500,28 +536,38 @@ __global__ void __launch_bounds__(kMmaThreads, 1) latent_attn_mma_kernel(const L
         *reinterpret_cast<float2*>(d + 8 * kPartPitch) = make_float2(sc[mt][b][2], sc[mt][b][3]);
       }
     __syncthreads();
+    if (tid == 0 && it > 0)                      // everyone is done with the tile before
+      for (int i = 2 * it + kMmaStages - 2; i < min(2 * it + kMmaStages, n_loads); ++i) load(i);
     {
       float s[KPT], mx = m;
 #pragma unroll
-      for (int i = 0; i < KPT; ++i) {
-        const int k = sub + TPR * i;
-        const float* d = part_s + row * kPartPitch + k;
-        s[i] = (d[0] + d[R * kPartPitch]) + (d[2 * R * kPartPitch] + d[3 * R * kPartPitch]);
-        s[i] = k < cnt ? s[i] * sl2 : -FLT_MAX;
-        mx = fmaxf(mx, s[i]);
+      for (int i = 0; i < KPT / 4; ++i) {
+        const int k = 4 * (sub + TPR * i);
+        float a[4][4];
+#pragma unroll
+        for (int x = 0; x < 4; ++x) load4(part_s + (x * R + row) * kPartPitch + k, a[x]);
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const float v = (a[0][e] + a[1][e]) + (a[2][e] + a[3][e]);
+          s[4 * i + e] = k + e < cnt ? v * sl2 : -FLT_MAX;
+          mx = fmaxf(mx, s[4 * i + e]);
+        }
       }
 #pragma unroll
       for (int o = TPR / 2; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
-      const float al = exp2f(m - mx);
+      const float al = ex2_approx(m - mx);     // a tile has at least one key: mx is a score
       m = mx;
       l *= al;
       if (sub == 0) alpha_s[row] = al;
 #pragma unroll
-      for (int i = 0; i < KPT; ++i) {
-        const int k = sub + TPR * i;
-        const float w = k < cnt ? exp2f(s[i] - mx) : 0.f;
-        l += w;
-        prob_s[row * kProbPitch + k] = __float2bfloat16_rn(w);
+      for (int i = 0; i < KPT / 4; ++i) {
+        float w[4];
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          w[e] = ex2_approx(s[4 * i + e] - mx);
+          l += w[e];
+        }
+        store4(prob_s + row * kProbPitch + 4 * (sub + TPR * i), w);
       }
     }
     __syncthreads();
@@ -546,51 +592,51 @@ __global__ void __launch_bounds__(kMmaThreads, 1) latent_attn_mma_kernel(const L
     }
 #pragma unroll
     for (int kk = 0; kk < kMmaKeys / 16; ++kk) {
+      if (kk * 16 >= cnt) continue;            // (rows that were not loaded are not numbers)
+      const uint32_t vrow = half[kk >> 1] + ((kk & 1) * 16 + (lt & 1) * 8 + lr) * 128;
       uint32_t pf[MT][4];
 #pragma unroll
       for (int mt = 0; mt < MT; ++mt)
         ldsm4(pf[mt], smem_u32(prob_s + (mt * 16 + (lt & 1) * 8 + lr) * kProbPitch + kk * 16 +
                                (lt >> 1) * 8));
+      uint32_t b[NP][4];
 #pragma unroll
       for (int j = 0; j < NP; ++j) {
-        const int pair = warp + 8 * j;
-        if (pair < n_pairs) {
-          uint32_t b[4];
-          ldsm4_t(b, smem_u32(tile + (kk * 16 + (lt & 1) * 8 + lr) * pitch + pair * 16 +
-                              (lt >> 1) * 8));
+        const int c8 = min(warp + 8 * j, n_pairs - 1) * 2 + (lt >> 1);
+        ldsm4_t(b[j], vrow + (c8 >> 3) * kMmaBlock + (((c8 ^ lr) & 7) << 4));
+      }
 #pragma unroll
-          for (int mt = 0; mt < MT; ++mt) {
-            mma16816(acc[mt][j][0], pf[mt], b[0], b[1]);
-            mma16816(acc[mt][j][1], pf[mt], b[2], b[3]);
-          }
+      for (int j = 0; j < NP; ++j)
+#pragma unroll
+        for (int mt = 0; mt < MT; ++mt) {
+          mma16816(acc[mt][j][0], pf[mt], b[j][0], b[j][1]);
+          mma16816(acc[mt][j][1], pf[mt], b[j][2], b[j][3]);
         }
+    }
+#pragma unroll
+    for (int x = 0; x < 2; ++x) {
+      st[x] += 2;
+      if (st[x] >= kMmaStages) {
+        st[x] -= kMmaStages;
+        ph[x] ^= 1;
       }
     }
-    __syncthreads();                             // everyone is done with this tile and the parts
-    if (warp == 0 && it + 2 < n_tiles) {
-      fence_proxy_async_smem();
-      load_tile(it + 2);
-    }
   }
-
-  if (abort_s) {                                 // bounded wait for copies still in flight
-    for (int it = max(n_tiles - 2, 0); it < n_tiles; ++it) {
-      const long long tq = clock64();
-      while (!mbar_try_wait(smem_u32(&full[it & 1]), (it >> 1) & 1))
-        if (clock64() - tq > kWaitLimitCycles / 8) break;
-    }
-    __syncthreads();
-  }
-
-  // the CTA's (m, l) and sums, then the cluster's: every CTA finishes its share of the columns
 #pragma unroll
   for (int o = TPR / 2; o > 0; o >>= 1) l += __shfl_xor_sync(0xffffffffu, l, o);
   if (sub == 0) {
     fin[row][0] = m;
     fin[row][1] = l;
   }
-  const int op = p.rank + 4;
-  float* out_s = reinterpret_cast<float*>(lat_b);
+  __syncthreads();                               // every stage has been read
+  if (abort_s) {                                 // bounded wait for copies still in flight
+    for (int i = max(n_loads - kMmaStages, 0); i < n_loads; ++i) {
+      const long long tq = clock64();
+      while (!mbar_try_wait(smem_u32(&full[i % kMmaStages]), (i / kMmaStages) & 1))
+        if (clock64() - tq > kWaitLimitCycles / 8) break;
+    }
+    __syncthreads();
+  }
 #pragma unroll
   for (int mt = 0; mt < MT; ++mt)
 #pragma unroll
@@ -604,54 +650,91 @@ __global__ void __launch_bounds__(kMmaThreads, 1) latent_attn_mma_kernel(const L
           *reinterpret_cast<float2*>(d + 8 * op) = make_float2(acc[mt][j][c][2], acc[mt][j][c][3]);
         }
       }
+
+  // the CTA's sums, then the cluster's: every CTA finishes its share of the columns
   if (p.splits > 1) cluster.sync();
   else __syncthreads();
-  const int vec = p.rank / 4, total = nr * vec;
-  const int per = (total + p.splits - 1) / p.splits;
-  for (int i = rank * per + tid; i < min(total, (rank + 1) * per); i += kMmaThreads) {
-    const int r = i / vec, d = (i - r * vec) * 4;
-    float o[4] = {0.f, 0.f, 0.f, 0.f}, ls = 0.f, mx = -FLT_MAX;
-    if (p.splits > 1) {
-      for (int k = 0; k < p.splits; ++k)
-        mx = fmaxf(mx, cluster.map_shared_rank(&fin[r][0], k)[0]);
-      for (int k = 0; k < p.splits; ++k) {
-        const float* f = cluster.map_shared_rank(&fin[r][0], k);
-        const float w = exp2f(f[0] - mx);
-        const float4 a = *reinterpret_cast<const float4*>(cluster.map_shared_rank(out_s, k) +
-                                                          r * op + d);
-        ls += w * f[1];
-        o[0] += w * a.x;
-        o[1] += w * a.y;
-        o[2] += w * a.z;
-        o[3] += w * a.w;
+  // a warp per head: lane k fetches (m, l) of CTA k, then the lanes walk the columns
+  T* out = static_cast<T*>(p.ol) + ((long long)t * p.H + h0) * p.rank;
+  for (int r = rank + p.splits * warp; r < nr; r += p.splits * (kMmaThreads / 32)) {
+    float mk = -FLT_MAX, lk = 0.f;
+    if (lane < p.splits) {
+      const float* f = cluster.map_shared_rank(&fin[r][0], lane);
+      mk = f[0];
+      lk = f[1];
+    }
+    const float w = exp2f(mk - warp_max(mk));
+    const float wn_ = w / warp_sum(w * lk);
+    constexpr int U = (NP * 128 + 127) / 128;    // 128 columns per pass of the warp
+    float4 o[U];
+#pragma unroll
+    for (int u = 0; u < U; ++u) o[u] = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 2
+    for (int k = 0; k < p.splits; ++k) {
+      const float* src = (p.splits > 1 ? cluster.map_shared_rank(out_s, k) : out_s) + r * op;
+      const float x = __shfl_sync(0xffffffffu, wn_, k);
+#pragma unroll
+      for (int u = 0; u < U; ++u) {
+        const int c = u * 128 + lane * 4;
+        if (c < p.rank) {
+          const float4 a = *reinterpret_cast<const float4*>(src + c);
+          o[u].x = fmaf(x, a.x, o[u].x);
+          o[u].y = fmaf(x, a.y, o[u].y);
+          o[u].z = fmaf(x, a.z, o[u].z);
+          o[u].w = fmaf(x, a.w, o[u].w);
+        }
       }
-    } else {
-      load4(out_s + r * op + d, o);
-      ls = fin[r][1];
     }
 #pragma unroll
-    for (int e = 0; e < 4; ++e) o[e] /= ls;
-    store4(static_cast<T*>(p.ol) + ((long long)t * p.H + h0 + r) * p.rank + d, o);
+    for (int u = 0; u < U; ++u) {
+      const int c = u * 128 + lane * 4;
+      if (c < p.rank) store4(out + (long long)r * p.rank + c, reinterpret_cast<const float*>(&o[u]));
+    }
   }
   if (p.splits > 1) cluster.sync();              // peers may still read this CTA's shared memory
 }
 
+// Rows of kd columns; a box brings kMmaRows of them, 64 columns wide, or (whole) all blocks of 64 columns
+// one after the other.
+static int latent_map(CUtensorMap* m, const void* base, int kd, long long rows, bool whole) {
+  EncodeTiledFn fn = flash_encode_fn();
+  if (!fn) return -10;
+  cuuint64_t dims[3] = {whole ? 64u : (cuuint64_t)kd, (cuuint64_t)rows,
+                        whole ? (cuuint64_t)(kd / 64) : 1u};
+  cuuint64_t strides[2] = {(cuuint64_t)kd * 2, whole ? 128u : (cuuint64_t)(rows * kd * 2)};
+  cuuint32_t box[3] = {64u, (cuuint32_t)kMmaRows, (cuuint32_t)dims[2]};
+  cuuint32_t estr[3] = {1u, 1u, 1u};
+  const CUresult r = fn(m, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, const_cast<void*>(base), dims,
+                        strides, box, estr, CU_TENSOR_MAP_INTERLEAVE_NONE,
+                        CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
+                        CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
+  return r == CUDA_SUCCESS ? 0 : -11;
+}
+
 template <int MT, int KQ, int NP, bool FUSED>
 static int latent_mma_launch(const LatentParams& p, cudaStream_t stream) {
-  const LatentPlan plan(p.rank + p.rot, p.rank, MT);
-  if (plan.total > 220 * 1024) return -2;
+  const int kd = p.rank + p.rot;
+  const LatentPlan plan(kd, p.rank, MT);
+  if (plan.total + 1024 > kMmaSmem) return -2;
+  // the cache as rows of kd columns
+  CUtensorMap tm;
+  const long long rows = (long long)p.slots * p.smax;
+  if (rows > 0x7fffffff) return -2;
+  const int boxes = kd % 64 ? (kd + 63) / 64 : 1;
+  const int r = latent_map(&tm, p.cache, kd, rows, kd % 64 == 0);
+  if (r) return r;
   auto kern = latent_attn_mma_kernel<MT, KQ, NP, FUSED>;
   static std::once_flag once;
   static cudaError_t err = cudaSuccess;
   std::call_once(once, [&] {
-    err = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024);
+    err = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, kMmaSmem);
   });
   if (err != cudaSuccess) return (int)err;
   cudaLaunchConfig_t cfg;
   memset(&cfg, 0, sizeof(cfg));
   cfg.gridDim = dim3(p.splits, (p.H + 16 * MT - 1) / (16 * MT), p.n);
   cfg.blockDim = dim3(kMmaThreads);
-  cfg.dynamicSmemBytes = plan.total;
+  cfg.dynamicSmemBytes = plan.total + 1024;      // alignment slack
   cfg.stream = stream;
   cudaLaunchAttribute attrs[2];
   int na = 0;
@@ -667,7 +750,7 @@ static int latent_mma_launch(const LatentParams& p, cudaStream_t stream) {
   }
   cfg.attrs = attrs;
   cfg.numAttrs = na;
-  return (int)cudaLaunchKernelEx(&cfg, kern, p);
+  return (int)cudaLaunchKernelEx(&cfg, kern, tm, boxes, p);
 }
 
 template <int MT>
@@ -675,6 +758,8 @@ static int latent_mma_pick(const LatentParams& p, bool fused, cudaStream_t s) {
   const int kd = p.rank + p.rot;
   if (kd <= 192 && p.rank <= 128)
     return fused ? latent_mma_launch<MT, 3, 1, true>(p, s) : latent_mma_launch<MT, 3, 1, false>(p, s);
+  if (kd <= 384 && p.rank <= 384)
+    return fused ? latent_mma_launch<MT, 6, 3, true>(p, s) : latent_mma_launch<MT, 6, 3, false>(p, s);
   return fused ? latent_mma_launch<MT, 9, 4, true>(p, s) : latent_mma_launch<MT, 9, 4, false>(p, s);
 }
 
