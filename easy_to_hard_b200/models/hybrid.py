@@ -501,6 +501,17 @@ def hybrid_config(d: Mapping) -> HybridConfig:
     return HYBRID_DESIGNS[name](d)
 
 
+def kernel_sources(cfg: HybridConfig) -> List[str]:
+    """Stems of the CUDA sources that a design's layers run on (all precisions)."""
+    names = {"gemm_umma", "gemm_persistent", "gemm_f32", "stream_norm"}
+    for L in cfg.layers:
+        names |= {"attention": {"attn_window", "flash_window"}, "gla": {"gla", "gla_chunk"},
+                  "latent": {"latent_attn", "flash_window"}}[L.mixer.kind]
+        if L.mlp is not None and L.mlp.kind == "moe":
+            names.add("moe")
+    return sorted(names)
+
+
 def config_in(folder: Union[str, Path]) -> Optional[dict]:
     """The parsed ``config.json`` of a checkpoint folder if it names one of the registered
     designs, else None (the folder then holds a gpt-fast checkpoint)."""

@@ -31,6 +31,7 @@ from __future__ import annotations
 
 from typing import Dict, Hashable, List, Optional, Sequence, Tuple
 
+import numpy as np
 import torch
 
 from ..ops import gemm, hybrid as hy
@@ -85,6 +86,12 @@ class _Scratch:
 
     def choice(self, n, top):
         return self._place[: n * top].view(n, top), self._ew[: n * top].view(n, top)
+
+
+def _positions(lengths, starts, slots):
+    """Position and cache slot of every packed token."""
+    return (np.concatenate([np.arange(a, a + n) for n, a in zip(lengths, starts)]),
+            np.repeat(slots, lengths))
 
 
 class HybridEngine(GenerationEngine):
@@ -184,14 +191,11 @@ class HybridEngine(GenerationEngine):
             if not cfg.parallel and f is not None:
                 hy.stream_norm(x, blk.norm2, h, eps=self.eps, offset=cfg.norm_offset)
                 tail = w.tail(n, blk.n_ff_tail)
-                self._count(1)
+                up = w.ff(n, blk.f_ff) if dense else None
+                self._count(1 + gemm.linear_packed(hw, blk.mat("w_ff"), up, bias=blk.b_ff,
+                                                   tail=tail, act_from=0, **dense))
                 if dense:
-                    up = w.ff(n, blk.f_ff)
-                    self._count(1 + gemm.linear_packed(hw, blk.mat("w_ff"), up, bias=blk.b_ff,
-                                                       tail=tail, act_from=0, **dense))
                     gemm.linear_residual_f32(up, blk.mat("w_down"), x)
-                else:
-                    gemm.linear_f32_out(hw, blk.mat("w_ff"), tail, bias=blk.b_ff)
                     self._count(1)
             if f is not None and f.kind == "moe":
                 pending = self._experts(w, blk, n, hw, tail)
@@ -234,6 +238,11 @@ class HybridEngine(GenerationEngine):
         cols = mix.p.H * mix.rank
         return (t[: n * cols].view(n, cols) for t in self._absorbed)
 
+    def _upload(self, *parts):
+        """int32 host sequences as slices of one device tensor."""
+        host = np.concatenate([np.asarray(p, dtype=np.int32) for p in parts])
+        return torch.from_numpy(host).to(self.dev).split([len(p) for p in parts])
+
     def _context(self, lengths, starts, slots) -> Optional[hy.LatentContext]:
         if self._latent is None:
             return None
@@ -255,7 +264,7 @@ class HybridEngine(GenerationEngine):
         """Runs the next tokens of open sequences. ``entries``: (key, token ids, places among
         these tokens whose logits are wanted). Returns the wanted logits, fp32 [wanted, vocab], in
         the order of the entries and places."""
-        toks, pos, slot, seg = [], [], [], [0]
+        toks, seg = [], [0]
         first: Dict[int, int] = {}       # entry -> its first packed token
         starts, slots = [], []
         keys = [k for k, _, _ in entries]
@@ -274,8 +283,6 @@ class HybridEngine(GenerationEngine):
             starts.append(at)
             slots.append(self.cache.slot(key))
             toks += [int(t) for t in ids]
-            pos += range(at, at + len(ids))
-            slot += [slots[-1]] * len(ids)
             seg.append(len(toks))
         rows = [first[i] + int(j) for i, (_, _, want) in enumerate(entries) for j in want]
         n = len(toks)
@@ -284,17 +291,16 @@ class HybridEngine(GenerationEngine):
             return out
         if min(toks) < 0 or max(toks) >= self.vocab:
             raise ValueError("token id outside the vocabulary")
-        longest = max(b - a for a, b in zip(seg, seg[1:]))
-        packed = torch.tensor(toks + pos + slot + seg + rows, dtype=torch.int32).to(self.dev)
-        t_d, p_d, s_d, seg_d, rows_d = packed.split([n, n, n, len(seg), len(rows)])
+        lengths = [b - a for a, b in zip(seg, seg[1:])]
+        alone = max(lengths) == 1
+        t_d, p_d, s_d, seg_d, rows_d = self._upload(
+            toks, *_positions(lengths, starts, slots), seg, rows)
         w = self._scratch if n <= self.B else _Scratch(self.model, n)
         hf = torch.zeros(len(rows), pad8(self.cfg.dim), dtype=self.model.dtype, device=self.dev)
         logits = torch.empty(len(rows), pad8(self.vocab), dtype=torch.float32, device=self.dev)
-        alone = longest == 1
         self._forward(w, n, t_d, p_d, s_d, rows=rows_d,
-                      seg=None if alone else (seg_d, len(seg) - 1, longest),
-                      ctx=None if alone else self._context([b - a for a, b in zip(seg, seg[1:])],
-                                                           starts, slots),
+                      seg=None if alone else (seg_d, len(lengths), max(lengths)),
+                      ctx=None if alone else self._context(lengths, starts, slots),
                       hf=hf, logits=logits)
         out.copy_(logits[:, : self.vocab])
         return out
@@ -389,29 +395,26 @@ class HybridEngine(GenerationEngine):
         self.prefill_launches = self.launches_per_step + 1
 
     def _prefill_part(self, ids, T, pads, slots, pick):
-        seg, cell, pos, slot, rows, fin = [0], [], [], [], [], []
+        seg, cell, rows, fin = [0], [], [], []
         pick = sorted(pick, key=lambda p: -p[2])
         for b, at, take in pick:
             lo = b * T + pads[b] + at
-            cell += range(lo, lo + take)
-            pos += range(at, at + take)
-            slot += [slots[b]] * take
-            seg.append(len(cell))
+            cell.append(np.arange(lo, lo + take))
+            seg.append(seg[-1] + take)
             if at + take == T - pads[b]:
-                rows.append(len(cell) - 1)
+                rows.append(seg[-1] - 1)
                 fin.append(b)
-        n = len(cell)
-        packed = torch.tensor(cell + pos + slot + seg + rows + fin, dtype=torch.int32).to(self.dev)
-        cell, pos, slot, seg_d, rows_d, fin_d = packed.split(
-            [n, n, n, len(seg), len(rows), len(fin)])
+        n = seg[-1]
+        lengths, starts = [t for _, _, t in pick], [a for _, a, _ in pick]
+        slots = [slots[b] for b, _, _ in pick]
+        ctx = self._context(lengths, starts, slots)
+        cell, pos, slot, seg_d, rows_d, fin_d = self._upload(
+            np.concatenate(cell), *_positions(lengths, starts, slots), seg, rows, fin)
         tokens = ids.reshape(-1)[cell.long()]
-        longest = max(t for _, _, t in pick)
         w = self._scratch if n <= self.B else _Scratch(self.model, n)
         whole = fin == list(range(ids.shape[0]))
         logits = self.logits if whole else torch.empty_like(self.logits)
-        ctx = self._context([t for _, _, t in pick], [a for _, a, _ in pick],
-                            [slots[b] for b, _, _ in pick])
-        self._forward(w, n, tokens, pos, slot, seg=(seg_d, len(seg) - 1, longest), ctx=ctx,
+        self._forward(w, n, tokens, pos, slot, seg=(seg_d, len(lengths), max(lengths)), ctx=ctx,
                       rows=rows_d, hf=self.hf, logits=logits)
         if not whole and fin:
             self.logits[fin_d.long()] = logits[: len(fin)]

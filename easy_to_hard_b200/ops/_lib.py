@@ -214,13 +214,23 @@ class NativeLibraryError(RuntimeError):
     pass
 
 
+_only = None
+
+
+def build_only(names) -> None:
+    """For programs that run a few kernels: unless the whole library is built already, ``lib()``
+    builds and loads one of these sources (stems of csrc/*.cu) alone."""
+    global _only
+    _only = tuple(names)
+
+
 @lru_cache(maxsize=1)
 def lib() -> C.CDLL:
     """Load (building first if the sources changed and nvcc is present) the native library."""
     path = _build.lib_path()
     try:
         if _build.needs_build():
-            path = _build.build()
+            path = _build.build(only=_only)
     except Exception as e:  # no nvcc on this machine: use the shipped binary if there is one
         if not path.exists():
             raise NativeLibraryError(f"native library missing and cannot be built: {e}") from e

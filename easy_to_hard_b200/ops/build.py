@@ -2,7 +2,9 @@
 
 Every ``csrc/*.cu`` file is compiled to an object and linked into
 ``easy_to_hard_b200/ops/_native/libe2h_b200.so``; the Python side loads it with ctypes
-(see ``_lib.py``). nvcc cross-compiles without a GPU, so this also runs on a CPU-only box.
+(see ``_lib.py``). nvcc cross-compiles without a GPU, so this also runs on a CPU-only box. An object
+is compiled again only when its source, a header or the flags have changed. A program that needs a
+few of the sources may build a library of these alone (``only``).
 
     python -m easy_to_hard_b200.ops.build [--force] [--verbose]
 """
@@ -16,6 +18,7 @@ import shutil
 import subprocess
 import sys
 from pathlib import Path
+from typing import Optional, Sequence
 
 HERE = Path(__file__).resolve().parent
 CSRC = HERE / "csrc"
@@ -46,19 +49,34 @@ def _digest(paths) -> str:
     return h.hexdigest()
 
 
-def lib_path() -> Path:
-    return OUT_DIR / LIB_NAME
+def sources(only: Optional[Sequence[str]] = None):
+    """All sources, or those whose stems ``only`` names."""
+    if only is None:
+        return sorted(CSRC.glob("*.cu"))
+    return [CSRC / f"{name}.cu" for name in sorted(set(only))]
 
 
-def sources():
-    return sorted(CSRC.glob("*.cu"))
+def _headers():
+    return [*CSRC.glob("*.cuh"), *CSRC.glob("*.h")]
 
 
-def needs_build() -> bool:
-    stamp = OUT_DIR / "build.stamp"
-    if not lib_path().exists() or not stamp.exists():
-        return True
-    return stamp.read_text().strip() != _digest(list(CSRC.glob("*.cu")) + list(CSRC.glob("*.cuh")))
+def lib_path(only: Optional[Sequence[str]] = None) -> Path:
+    if only is None:
+        return OUT_DIR / LIB_NAME
+    tag = hashlib.sha256(" ".join(sorted(set(only))).encode()).hexdigest()[:8]
+    return OUT_DIR / f"libe2h_part_{tag}.so"
+
+
+def _stamp_path(only: Optional[Sequence[str]] = None) -> Path:
+    return OUT_DIR / "build.stamp" if only is None else lib_path(only).with_suffix(".stamp")
+
+
+def _fresh(path: Path, stamp: Path, digest: str) -> bool:
+    return path.exists() and stamp.exists() and stamp.read_text().strip() == digest
+
+
+def needs_build(only: Optional[Sequence[str]] = None) -> bool:
+    return not _fresh(lib_path(only), _stamp_path(only), _digest(sources(only) + _headers()))
 
 
 def build_phase_clock() -> Path:
@@ -75,51 +93,59 @@ def build_phase_clock() -> Path:
     return out
 
 
-def build(force: bool = False, verbose: bool = False) -> Path:
+def build(force: bool = False, verbose: bool = False,
+          only: Optional[Sequence[str]] = None) -> Path:
     """Compile and link; returns the path of the shared library. Processes that start together
     (one per GPU under torchrun) take a file lock, so one of them builds and the others find the
     finished library."""
-    if not force and not needs_build():
-        return lib_path()
+    if not force and not needs_build(only):
+        return lib_path(only)
     OUT_DIR.mkdir(parents=True, exist_ok=True)
     import fcntl
     with open(OUT_DIR / "build.lock", "w") as lock:
         fcntl.flock(lock, fcntl.LOCK_EX)
         try:
-            if not force and not needs_build():     # another process built it meanwhile
-                return lib_path()
-            return _build_locked(verbose)
+            if not force and not needs_build(only):     # another process built it meanwhile
+                return lib_path(only)
+            return _build_locked(force, verbose, only)
         finally:
             fcntl.flock(lock, fcntl.LOCK_UN)
 
 
-def _build_locked(verbose: bool) -> Path:
+def _build_locked(force: bool, verbose: bool, only: Optional[Sequence[str]]) -> Path:
     nvcc = _nvcc()
-    srcs = sources()
+    srcs = sources(only)
     extra = ["-Xptxas", "-v"] if verbose else []
 
     def compile_one(src: Path) -> Path:
-        obj = OUT_DIR / (src.stem + ".o")
+        obj, stamp = OUT_DIR / (src.stem + ".o"), OUT_DIR / (src.stem + ".stamp")
+        digest = _digest([src] + _headers())
+        if not force and not verbose and _fresh(obj, stamp, digest):
+            return obj
         cmd = [nvcc, *NVCC_FLAGS, *extra, "-I", str(CSRC), "-c", str(src), "-o", str(obj)]
         r = subprocess.run(cmd, capture_output=True, text=True)
         if verbose or r.returncode != 0:
             sys.stderr.write(f"--- {src.name}\n{r.stdout}{r.stderr}\n")
         if r.returncode != 0:
             raise RuntimeError(f"nvcc failed on {src.name}")
+        stamp.write_text(digest)
         return obj
 
+    digest = _digest(srcs + _headers())
+    # the slowest sources first
+    srcs = sorted(srcs, key=lambda p: -p.stat().st_size)
     with cf.ThreadPoolExecutor(max_workers=min(8, len(srcs))) as ex:
         objs = list(ex.map(compile_one, srcs))
-    tmp = OUT_DIR / (LIB_NAME + ".tmp")
+    out = lib_path(only)
+    tmp = out.with_suffix(".so.tmp")
     cmd = [nvcc, "-shared", "-o", str(tmp), *[str(o) for o in objs],
            "-gencode", "arch=compute_100a,code=sm_100a"]
     r = subprocess.run(cmd, capture_output=True, text=True)
     if r.returncode != 0:
         raise RuntimeError(f"link failed:\n{r.stdout}{r.stderr}")
-    os.replace(tmp, lib_path())
-    (OUT_DIR / "build.stamp").write_text(
-        _digest(list(CSRC.glob("*.cu")) + list(CSRC.glob("*.cuh"))))
-    return lib_path()
+    os.replace(tmp, out)
+    _stamp_path(only).write_text(digest)
+    return out
 
 
 if __name__ == "__main__":

@@ -503,8 +503,16 @@ def _gemm_f32(a, b, *, epi, out, a2=None, aux=None, bias=None, act_from=None, ta
 def linear_packed(x, w, out, *, bias=None, act_from=None, tail=None, act: str = "relu2") -> int:
     """Several projections of x at once: ``out`` [T, F0] takes the first F0 features of ``w`` in
     x's type (activation ``act`` from feature ``act_from`` on), ``tail`` [T, F - F0] the others in
-    fp32; ``bias`` fp32 [F]. Returns the number of launches."""
-    F0, F = out.shape[1], w.shape[0]
+    fp32; ``bias`` fp32 [F]. ``out`` None: the tail is all. Returns the number of launches."""
+    F0, F = 0 if out is None else out.shape[1], w.shape[0]
+    if F0 == 0:
+        if x.dtype == torch.float32:
+            _gemm_f32(w, x, epi=EPI_STORE_F32, out=tail, bias=bias)
+        elif bias is None and x.shape[0] > 128:
+            linear_rows(x, w, tail)
+        else:
+            gemm(w, x, epi=EPI_STORE_F32, out=tail, bias=bias)
+        return 1
     if x.dtype == torch.float32:
         _gemm_f32(w, x, epi=EPI_STORE_F32, out=out, bias=bias, act_from=act_from, tail=tail,
                   tail_from=F0 if F > F0 else 0, act=act)
@@ -517,8 +525,20 @@ def linear_packed(x, w, out, *, bias=None, act_from=None, tail=None, act: str = 
     if F == F0:
         return 1
     # many tokens: the few tail features would break the large tiles of the main product
-    gemm(w[F0:], x, epi=EPI_STORE_F32, out=tail, bias=None if bias is None else bias[F0:])
+    if bias is None:
+        linear_rows(x, w[F0:], tail)
+    else:
+        gemm(w[F0:], x, epi=EPI_STORE_F32, out=tail, bias=bias[F0:])
     return 2
+
+
+def linear_rows(x, w, out) -> None:
+    """out = x @ w^T with the tokens on the tensor-memory lanes: a thread of the epilogue owns one
+    token and writes its features as vectors. For many tokens and a short contraction, where the
+    epilogue of a tile takes longer than its main loop, or few features, where the tokens give more
+    tiles. bf16 operands; out bf16 or fp32."""
+    gemm(x, w, epi=EPI_ROWMAJOR_BF16 if out.dtype == torch.bfloat16 else EPI_ROWMAJOR_F32_ACC,
+         out=out)
 
 
 def linear_residual_f32(x, w, residual) -> None:
@@ -529,10 +549,9 @@ def linear_residual_f32(x, w, residual) -> None:
         gemm(w, x, epi=EPI_RESIDUAL_F32, out=residual, aux=residual)
 
 
-def linear_f32_out(x, w, out, scale: float = 1.0, softcap: float = 0.0, bias=None) -> None:
-    """out (fp32) = (x @ w^T + bias) * scale, then softcap * tanh(out / softcap) unless ``softcap`` is
-    0."""
-    kw = dict(epi=EPI_STORE_F32, out=out, out_scale=scale, softcap=softcap, bias=bias)
+def linear_f32_out(x, w, out, scale: float = 1.0, softcap: float = 0.0) -> None:
+    """out (fp32) = x @ w^T * scale, then softcap * tanh(out / softcap) unless ``softcap`` is 0."""
+    kw = dict(epi=EPI_STORE_F32, out=out, out_scale=scale, softcap=softcap)
     _gemm_f32(w, x, **kw) if x.dtype == torch.float32 else gemm(w, x, **kw)
 
 

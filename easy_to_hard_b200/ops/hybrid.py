@@ -6,6 +6,7 @@ from __future__ import annotations
 import ctypes as C
 from typing import Optional
 
+import numpy as np
 import torch
 
 from . import _lib, gemm
@@ -162,23 +163,24 @@ class LatentContext:
         slot. ``window``: the widest of the layers (0: unlimited)."""
         self.n_long = self.n_long_seg = self.seg_max = self.n_ctx = 0
         self.src = self.pos = self.slot = self.shift = None
-        src, pos, slot, shift, at = [], [], [], [], 0
+        src, pos, slot, shift = [], [], [], []
         for n, p0, s in zip(lengths, starts, slots):
             lo = max(p0 - window + 1, 0) if window else 0
             if not expand or not LatentAttention.expands(n, p0 - lo):
                 break
-            shift.append(len(src) - lo)
-            src += [-1] * (p0 - lo) + list(range(at, at + n))
-            pos += range(lo, p0 + n)
-            slot += [s] * (p0 + n - lo)
-            at += n
+            shift.append(self.n_ctx - lo)
+            src += [np.full(p0 - lo, -1), np.arange(self.n_long, self.n_long + n)]
+            pos.append(np.arange(lo, p0 + n))
+            slot.append(np.full(p0 + n - lo, s))
+            self.n_long += n
+            self.n_ctx += p0 + n - lo
             self.n_long_seg += 1
             self.seg_max = max(self.seg_max, n)
-        self.n_long, self.n_ctx = at, len(src)
         if src:
             m = self.n_ctx
-            d = torch.tensor(src + pos + slot + shift, dtype=torch.int32).to(device)
-            self.src, self.pos, self.slot, self.shift = d.split([m, m, m, len(shift)])
+            d = np.concatenate(src + pos + slot + [shift]).astype(np.int32)
+            self.src, self.pos, self.slot, self.shift = torch.from_numpy(d).to(device).split(
+                [m, m, m, len(shift)])
 
 
 class LatentAttention:
@@ -270,7 +272,7 @@ class LatentAttention:
 
     def expand(self, rows, kv) -> None:
         """Keys [H x dim] and values [H x vdim] of the context rows."""
-        gemm.linear(rows[:, : self.rank], self.w_kv, out=kv)
+        gemm.linear_rows(rows[:, : self.rank], self.w_kv, kv)
 
     def flash(self, act, pos, slot, seg, ctx: LatentContext, rows, kv) -> None:
         p = self._bind(act, pos, slot)

@@ -31,8 +31,11 @@ def main(argv: Optional[Sequence[str]] = None, lines=None) -> int:
                     help="positions the cache is built for")
     a = ap.parse_args(argv)
     from .models.engine import get_engine
-    from .models.hybrid import load_hybrid
+    from .models.hybrid import config_in, hybrid_config, kernel_sources, load_hybrid
     from .ops import _lib
+    cfg = config_in(a.model)
+    if cfg is not None:
+        _lib.build_only(kernel_sources(hybrid_config(cfg)))
     model = load_hybrid(a.model, "cuda", getattr(torch, a.dtype))
     eng = get_engine(model, SLOTS, max(a.max_tokens, 1), use_graph=False)
     for line in (sys.stdin if lines is None else lines):

@@ -153,3 +153,25 @@ def test_window_of_the_oracle():
     v = O.visible(12, 4)
     assert v[9].tolist() == [False] * 6 + [True] * 4 + [False] * 2
     assert v[2].tolist() == [True] * 3 + [False] * 9 and O.visible(5, None).sum() == 15
+
+
+def test_sources_of_a_design_are_those_its_layers_run_on():
+    """What a fresh checkout compiles before it replays a trace: the named sources exist, define the
+    entry points the layers call, and depend on no other source."""
+    import re
+
+    import bovinex_models as B
+    from easy_to_hard_b200.models.hybrid import hybrid_config, kernel_sources
+    from easy_to_hard_b200.ops import build
+    names = kernel_sources(hybrid_config(M.ZOO["mixed"]))
+    assert "latent_attn" in names and "moe" in names
+    assert not {"attn_window", "gla", "gla_chunk", "loss", "flash_attn"} & set(names)
+    bare = kernel_sources(hybrid_config(M.config([M.layer()])))
+    assert "moe" not in bare
+    assert {"attn_window", "gla", "moe"} <= set(kernel_sources(hybrid_config(B.ZOO["mixed"])))
+    srcs = build.sources(names)
+    assert all(s.is_file() for s in srcs)
+    entry = set(re.findall(r'extern "C" int (e2h_\w+)', "".join(s.read_text() for s in srcs)))
+    assert {"e2h_gemm_umma", "e2h_gemm_persistent", "e2h_gemm_f32", "e2h_stream_norm",
+            "e2h_moe_route", "e2h_latent_prep", "e2h_latent_attn", "e2h_flash_window"} <= entry
+    assert build.lib_path(names) != build.lib_path() != build.lib_path(bare)

@@ -69,6 +69,9 @@ def test_projection_with_gelu(dt, T, K, F, tail):
     _close(out, O.gelu(y[:, :F]), _tol(dtype, 2e-6, 5e-3))
     if tail:
         _close(tl[:, :tail], y[:, F:], 1e-5)
+        for bias in (None, torch.randn(tail, generator=g).cuda()):      # nothing but a tail
+            gemm.linear_packed(x[:, :K], w[F:, :K], None, tail=tl, bias=bias)
+            _close(tl[:, :tail], y[:, F:] + (0 if bias is None else bias), 1e-5)
     _ok()
 
 
