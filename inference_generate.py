@@ -12,7 +12,7 @@ under an exclusive ``flock`` (tensor-parallel rank 0 of each group writes). ``--
 skips the (idx, sample) pairs already present in the output file.
 
 ``--checkpoint_path DIR/model.safetensors`` with a ``DIR/config.json`` that names a hybrid design
-(``models.hybrid``: Bovinex) runs that design; everything else stays the same.
+(``models.hybrid``: Bovinex, Ruralorn) runs that design; everything else stays the same.
 
 On CUDA, ``generate`` runs on the ``DecodeEngine`` (CUDA-graph decode over the sm_100a kernels,
 static KV cache sized to prompt + new tokens instead of the whole ``block_size``); ``--compile``
