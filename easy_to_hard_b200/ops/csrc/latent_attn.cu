@@ -308,12 +308,12 @@ __device__ __forceinline__ uint32_t tile_at(uint32_t tile, int r, int c) {
 // MT: blocks of 16 query heads; KQ: 16-column steps of a row per warp (a quarter of the row); NP: pairs
 // of 8-column tiles of the latent per warp.
 //
-// TMA fills the ring 32 rows at a time (rows past the last key are read and masked), a stage as soon as
-// every warp is past the tile that read it last. Work of the eight warps on a tile of 64 keys: scores - warp (quarter of the columns,
-// half of the keys), its query fragments stay in registers; the four partial scores of a (head, key)
-// meet in shared memory, where 256 / R threads run the softmax of a head; output - warp (1/8 of the
-// latent columns, all keys). Every byte of a cache row is read twice from shared memory, once per
-// product. Two barriers per tile.
+// TMA fills the ring 32 rows at a time (rows past the last key are read and masked), a stage as soon
+// as every warp is past the tile that read it last. Work of the eight warps on a tile of 64 keys:
+// scores - warp (quarter of the columns, half of the keys), its query fragments stay in registers; the
+// four partial scores of a (head, key) meet in shared memory, where 256 / R threads run the softmax of
+// a head; output - warp (1/8 of the latent columns, all keys). Every byte of a cache row is read twice
+// from shared memory, once per product. Two barriers per tile.
 template <int MT, int KQ, int NP, bool FUSED>
 __global__ void __launch_bounds__(kMmaThreads, 1)
 latent_attn_mma_kernel(const __grid_constant__ CUtensorMap tm, const int boxes,
@@ -456,7 +456,7 @@ latent_attn_mma_kernel(const __grid_constant__ CUtensorMap tm, const int boxes,
   const int s_begin = kq * per_q, s_count = max(0, min(per_q, ks - s_begin));
   const int c8_last = ks * 2 - 2;                // steps past the row repeat its end, times zero
   uint32_t qf[KQ][MT][4];
-  const int lr = lane & 7, lt = lane >> 3;     // row and tile of this lane's ldmatrix address
+  const int lr = lane & 7, lt = lane >> 3;       // row and tile of this lane's ldmatrix address
 #pragma unroll
   for (int s = 0; s < KQ; ++s)
 #pragma unroll
